@@ -6,24 +6,6 @@
 // points, see SURVEY.md §7 "bit-level parity traps".
 #include "common.cuh"
 
-// Mirrors of the approximate ops Triton emits for the reference kernels on sm_100a
-// (probed: sqrt.approx.ftz.f32, div.full.f32, ex2.approx) so results round the same way.
-__device__ __forceinline__ float sqrt_approx(float x) {
-  float r;
-  asm("sqrt.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(x));
-  return r;
-}
-__device__ __forceinline__ float div_full(float a, float b) {
-  float r;
-  asm("div.full.f32 %0, %1, %2;" : "=f"(r) : "f"(a), "f"(b));
-  return r;
-}
-__device__ __forceinline__ float ex2_approx(float x) {
-  float r;
-  asm("ex2.approx.f32 %0, %1;" : "=f"(r) : "f"(x));
-  return r;
-}
-
 // --------------------------------------------------------------------------- //
 // skip_rmsnorm  (reference: lite_llama/kernels/skip_rmsnorm.py:126-234)
 //   r += x (stored back in the activation dtype), y = round(r_f32 * rrms) * w
@@ -75,7 +57,7 @@ __global__ void __launch_bounds__(512) skip_rmsnorm_block_kernel(T* __restrict__
   float tot = 0.f;
   const int nw = blockDim.x >> 5;
   for (int i = 0; i < nw; ++i) tot += red[i];
-  const float rrms = div_full(1.0f, sqrt_approx(tot / (float)n + eps));
+  const float rrms = 1.0f / sqrtf(tot / (float)n + eps);
 #pragma unroll
   for (int i = 0; i < VPT_MAX; ++i) {
     const int c = threadIdx.x + i * blockDim.x;
@@ -114,7 +96,7 @@ __global__ void skip_rmsnorm_warp_kernel(T* __restrict__ y, const T* __restrict_
     ss += s * s;
   }
   ss = warp_reduce_sum(ss);
-  const float rrms = div_full(1.0f, sqrt_approx(ss / (float)n + eps));
+  const float rrms = 1.0f / sqrtf(ss / (float)n + eps);
   for (int64_t c = lane; c < n; c += 32) {
     float s = to_f32(xr[c]);
     if (rr) {
@@ -156,7 +138,7 @@ __global__ void skip_rmsnorm_warp_reg_kernel(T* __restrict__ y, const T* __restr
     }
   }
   ss = warp_reduce_sum(ss);
-  const float rrms = div_full(1.0f, sqrt_approx(ss / (float)n + eps));
+  const float rrms = 1.0f / sqrtf(ss / (float)n + eps);
 #pragma unroll
   for (int i = 0; i < KEEP; ++i) {
     const int64_t c = lane + 32 * i;
@@ -231,7 +213,6 @@ extern "C" int b2l_skip_rmsnorm(void* y, const void* x, void* residual, const vo
 // rope_emb_forward (reference: lite_llama/kernels/rope_emb.py:14-134)
 //   half-split rotation, in place, arithmetic in the activation dtype:
 //     new1 = fma(x1, cos, -(x2*sin));  new2 = fma(x2, cos, x1*sin)
-//   (exactly the mul+fma contraction Triton emits for this kernel on sm_100a)
 // --------------------------------------------------------------------------- //
 __device__ __forceinline__ void rope_pair(__half2& a, __half2& b, __half2 c, __half2 s) {
   __half2 t1 = __hmul2(b, s);
@@ -437,9 +418,8 @@ extern "C" int b2l_rope_kv_write(void* q, void* k, const void* v, const void* co
 // the `b` pointer offset / row strides (gate and up halves of one row).
 // --------------------------------------------------------------------------- //
 __device__ __forceinline__ float silu_f32(float x) {
-  // sigmoid = 1 / (1 + exp(-x)) with ex2.approx + div.full, as Triton lowers tl.sigmoid
-  const float e = ex2_approx(-x * 1.4426950408889634f);
-  return x * div_full(1.0f, 1.0f + e);
+  // the fast intrinsics' error is far below the rounding of the 16-bit result
+  return __fdividef(x, 1.0f + __expf(-x));
 }
 
 template <typename T>
@@ -587,7 +567,7 @@ extern "C" int b2l_update_kv_index(void* table, const void* b_req_idx, int req_w
 // --------------------------------------------------------------------------- //
 // Per-token dynamic int8 activation quantisation
 // (reference: lite_llama/kernels/quantization/w8a8.py:35-68)
-//   scale = absmax/127 (1.0 if 0);  q = trunc_toward_zero(x / scale)   [div.full.f32 + cvt.rzi]
+//   scale = absmax/127 (1.0 if 0);  q = trunc_toward_zero(x / scale)
 // One CTA per row, row kept in registers (single HBM pass instead of the reference's two).
 // --------------------------------------------------------------------------- //
 template <typename T>
@@ -606,14 +586,10 @@ __global__ void __launch_bounds__(256) quantize_act_int8_kernel(int8_t* __restri
   __syncthreads();
   float m = 0.f;
   for (int i = 0; i < (int)(blockDim.x >> 5); ++i) m = fmaxf(m, red[i]);
-  float scale = div_full(m, 127.0f);
+  float scale = m / 127.0f;
   scale = scale > 0.f ? scale : 1.0f;
   for (int64_t i = threadIdx.x; i < k; i += blockDim.x) {
-    const float v = div_full(to_f32(xr[i]), scale);
-    int32_t iv;
-    // Triton's fp32 -> int8 cast: cvt.rzi (truncate toward zero), then narrow.
-    asm("cvt.rzi.s32.f32 %0, %1;" : "=r"(iv) : "f"(v));
-    qr[i] = (int8_t)iv;
+    qr[i] = (int8_t)__float2int_rz(to_f32(xr[i]) / scale);      // truncates toward zero, then narrows
   }
   if (threadIdx.x == 0) scales[row] = scale;
 }
@@ -689,7 +665,7 @@ __global__ void __launch_bounds__(512) skip_rmsnorm_quant_kernel(int8_t* __restr
   float tot = 0.f;
   const int nw = blockDim.x >> 5;
   for (int i = 0; i < nw; ++i) tot += red[i];
-  const float rrms = div_full(1.0f, sqrt_approx(tot / (float)n + eps));
+  const float rrms = 1.0f / sqrtf(tot / (float)n + eps);
   // the norm output, rounded to the activation dtype exactly like the stand-alone kernel, stays in registers
   float amax = 0.f;
 #pragma unroll
@@ -712,7 +688,7 @@ __global__ void __launch_bounds__(512) skip_rmsnorm_quant_kernel(int8_t* __restr
   __syncthreads();
   float m = 0.f;
   for (int i = 0; i < nw; ++i) m = fmaxf(m, red_max[i]);
-  float scale = div_full(m, 127.0f);
+  float scale = m / 127.0f;
   scale = scale > 0.f ? scale : 1.0f;
 #pragma unroll
   for (int i = 0; i < VPT_MAX; ++i) {
@@ -721,9 +697,7 @@ __global__ void __launch_bounds__(512) skip_rmsnorm_quant_kernel(int8_t* __restr
       uint32_t lo = 0u, hi = 0u;
 #pragma unroll
       for (int j = 0; j < 8; ++j) {
-        int32_t iv;
-        asm("cvt.rzi.s32.f32 %0, %1;" : "=r"(iv) : "f"(div_full(vals[i][j], scale)));   // Triton's fp32 -> int8 cast
-        const uint32_t b = (uint32_t)(uint8_t)(int8_t)iv;
+        const uint32_t b = (uint32_t)(uint8_t)(int8_t)__float2int_rz(vals[i][j] / scale);
         if (j < 4) lo |= b << (8 * j); else hi |= b << (8 * (j - 4));
       }
       *reinterpret_cast<uint2*>(qr + c * 8) = make_uint2(lo, hi);

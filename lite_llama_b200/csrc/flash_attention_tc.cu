@@ -2,8 +2,8 @@
 //
 // Replaces lite_llama/kernels/flashattention2_nopad.py:45-231 for the shapes the decoder uses (D = 128, heads packed
 // inside a token row); same contract as flash_attention_nopad.cu, which stays the path for other head sizes.
-// The reference's Triton build already lowers this op to tcgen05.mma on sm_100a, so the legacy
-// mma.sync kernel lost to it 2x (profiles/r2c_triton_vs_b200.md); this kernel is the B200-native one.
+// The mma.sync kernel measured twice the reference's time at these shapes (profiles/r2c_triton_vs_b200.md); this
+// kernel is the B200-native one.
 //
 // One CTA = 128 query rows of one (sequence, q head), 192 threads:
 //   warp 0      loader: Q once, then 128-key K and V tiles through separate 3-deep rings (2-D TMA, 128B swizzle;

@@ -8,7 +8,7 @@
 // B200 design (DESIGN.md "flash_decoding"):
 //  * one CTA per (split, kv-head block, batch row) streams WHOLE TOKEN ROWS: in the fused pool a
 //    token's K heads and V heads are one contiguous 2*Hkv*D*2-byte run (4 KiB for Llama-3-8B), so a
-//    single 1-D bulk async copy (cp.async.bulk -> SASS UBLKCP, the TMA engine) per token brings in
+//    single 1-D bulk async copy (cp.async.bulk, the TMA engine) per token brings in
 //    everything every head needs.  (First version: one CTA per kv head with 256-byte copies reached
 //    only 29 % of HBM peak -- the copy engine's request rate, not bytes, was the limit.)
 //  * a dedicated producer warp walks the token table and issues the copies into a 3-4 stage

@@ -268,17 +268,8 @@ __device__ __forceinline__ void umma_f16_ts(uint32_t tmem_d, uint32_t tmem_a, ui
       ::"r"(tmem_d), "r"(tmem_a), "l"(bdesc), "r"(idesc), "r"(accumulate) : "memory");
 }
 
-// same approximate ops as elementwise.cu's swiglu (Triton's lowering of tl.sigmoid on sm_100a)
-__device__ __forceinline__ float ex2_approx_q(float x) {
-  float r;
-  asm("ex2.approx.f32 %0, %1;" : "=f"(r) : "f"(x));
-  return r;
-}
-__device__ __forceinline__ float div_full_q(float a, float b) {
-  float r;
-  asm("div.full.f32 %0, %1, %2;" : "=f"(r) : "f"(a), "f"(b));
-  return r;
-}
+// the swiglu kernel's SiLU (csrc/elementwise.cu), so the fused epilogue rounds like the unfused path
+__device__ __forceinline__ float silu_q(float x) { return __fdividef(x, 1.0f + __expf(-x)); }
 __device__ __forceinline__ float lds_f32(const float* p) {
   float v;
   asm volatile("ld.shared.f32 %0, [%1];" : "=f"(v) : "r"(smem_u32(p)));
@@ -962,8 +953,7 @@ gemm_quant_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_const
             const float other = __shfl_xor_sync(0xffffffffu, mine, 1);
             const int m = m_tile * BT + j;
             if (n_ok && (epi_tid & 1) == 0 && m < p.M) {
-              const float e = ex2_approx_q(-mine * 1.4426950408889634f);
-              const float sl = mine * div_full_q(1.0f, 1.0f + e);
+              const float sl = silu_q(mine);
               y[(int64_t)m * p.ldy + (n >> 1)] = __float2half_rn(sl * other);
             }
           }
@@ -1352,8 +1342,7 @@ gemm_quant_kernel(const __grid_constant__ CUtensorMap tmap_w, const __grid_const
           const float mine = __half2float(__float2half_rn(sum[i] + bv));
           const float other = __shfl_xor_sync(0xffffffffu, mine, 1);
           if (n_ok && (n_local & 1) == 0 && m < p.M) {
-            const float e = ex2_approx_q(-mine * 1.4426950408889634f);
-            yy[(int64_t)m * p.ldy + (n >> 1)] = __float2half_rn(mine * div_full_q(1.0f, 1.0f + e) * other);
+            yy[(int64_t)m * p.ldy + (n >> 1)] = __float2half_rn(silu_q(mine) * other);
           }
         } else if (n_ok && m < p.M) {
           yy[(int64_t)m * p.ldy + n] = __float2half_rn(sum[i] + bv);

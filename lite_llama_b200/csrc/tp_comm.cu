@@ -74,16 +74,6 @@ __device__ __forceinline__ uint4 ld_pkt(const void* p) {
   asm volatile("ld.volatile.global.v4.u32 {%0,%1,%2,%3}, [%4];" : "=r"(v.x), "=r"(v.y), "=r"(v.z), "=r"(v.w) : "l"(p) : "memory");
   return v;
 }
-__device__ __forceinline__ float sqrt_approx_f(float x) {
-  float r;
-  asm("sqrt.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(x));
-  return r;
-}
-__device__ __forceinline__ float div_full_f(float a, float b) {
-  float r;
-  asm("div.full.f32 %0, %1, %2;" : "=f"(r) : "f"(a), "f"(b));
-  return r;
-}
 template <typename T> __device__ __forceinline__ void unpack2(uint32_t w, float& a, float& b) {
   const T* e = reinterpret_cast<const T*>(&w);
   a = to_f32(e[0]); b = to_f32(e[1]);
@@ -213,7 +203,7 @@ __global__ void __launch_bounds__(kThreads) tp_allreduce_rmsnorm_kernel(const Fu
   float tot = 0.f;
 #pragma unroll
   for (int i = 0; i < kThreads / 32; ++i) tot += red[i];
-  const float rrms = div_full_f(1.0f, sqrt_approx_f(tot / (float)p.n + p.eps));
+  const float rrms = 1.0f / sqrtf(tot / (float)p.n + p.eps);
   const uint32_t* ww = reinterpret_cast<const uint32_t*>(p.w);
   uint32_t* yw = reinterpret_cast<uint32_t*>(yr);
 #pragma unroll
