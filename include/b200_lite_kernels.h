@@ -284,40 +284,43 @@ int b2l_gelu(void* out, const void* x, int64_t total, int tanh_form, int dtype, 
 /* out_f32 = cap * tanh(scale * x / cap) (cap <= 0: scale * x) as fp32: scaled, soft-capped logits. */
 int b2l_softcap_to_f32(void* out_f32, const void* x, int64_t total, float cap, float scale, int dtype, void* stream);
 /* y[t, h, :] = W[h] . x[t, h, :] for W [heads, n, k] (csrc/gemm_simt.cu); x / y rows hold the heads side by side
- * (strides in elements); gate (nullable) [m, >= heads]: y[t, h, :] *= sigmoid(gate[t, h]). */
+ * (strides in elements); gate (nullable) [m, >= heads]: y[t, h, :] *= sigmoid(gate[t, h]); with gate_elements it is
+ * [m, >= heads * n]: y[t, h, c] *= sigmoid(gate[t, h * n + c]). */
 int b2l_head_linear(void* y, int64_t y_row_stride, int64_t y_head_stride, const void* x, int64_t x_row_stride,
-                    int64_t x_head_stride, const void* w, const void* gate, int64_t gate_row_stride, int64_t m,
-                    int heads, int64_t n, int64_t k, int dtype, void* stream);
+                    int64_t x_head_stride, const void* w, const void* gate, int64_t gate_row_stride, int gate_elements,
+                    int64_t m, int heads, int64_t n, int64_t k, int dtype, void* stream);
 /* Grouped product over expert-sorted slots (b2l_moe_align_block_size with block_size = b2l_moe_gemm_simt_block()):
- * c[s, :] = act(W[expert(s)] . a[s / top_k, :]) * slot_weight_f32[s] (nullable); act 0 = none, 1 = exact gelu;
- * W [experts, n, k] dense; every dtype of this section, fp32 sums in ascending k. */
+ * c[s, :] = act(W[expert(s)] . a[s / top_k, :]) * slot_weight_f32[s] (nullable); act 0 = none, 1 = exact gelu,
+ * 2 = the clamped gated unit of interleaved rows (2i = gate i, 2i + 1 = up i, n / 2 output columns):
+ * g' sigmoid(alpha g') (u' + 1), g' = min(g, limit), u' = clamp(u, -limit, limit); W [experts, n, k] dense; every dtype of this section, fp32 sums in ascending k. */
 int b2l_moe_gemm_simt_block(void);
 int b2l_moe_gemm_simt(void* c, const void* a, const void* w, const void* slot_weight_f32,
                       const void* sorted_token_ids, const void* expert_ids, const void* num_tokens_post_padded,
                       int64_t em, int64_t num_valid_slots, int top_k, int64_t n, int64_t k, int64_t a_row_stride,
-                      int64_t c_row_stride, int act, int dtype, void* stream);
+                      int64_t c_row_stride, int act, float limit, float alpha, int dtype, void* stream);
 /* Tensor-core (mma.sync, fp32 accumulators) versions of b2l_head_linear and b2l_moe_gemm_simt for 16-bit dtypes
  * (csrc/gemm_rows_mma.cu); b2l_rows_gemm_mma_ok says whether they take the operands (k and the x strides multiples
  * of 8 elements, 16-byte aligned bases).  b2l_moe_gemm_mma: block_size 16, 64 or 128 = the block size of the alignment. */
 int b2l_rows_gemm_mma_ok(const void* x, const void* w, int64_t k, int64_t x_row_stride, int64_t x_head_stride,
                          int dtype);
 int b2l_head_linear_mma(void* y, int64_t y_row_stride, int64_t y_head_stride, const void* x, int64_t x_row_stride,
-                        int64_t x_head_stride, const void* w, const void* gate, int64_t gate_row_stride, int64_t m,
-                        int heads, int64_t n, int64_t k, int dtype, void* stream);
+                        int64_t x_head_stride, const void* w, const void* gate, int64_t gate_row_stride,
+                        int gate_elements, int64_t m, int heads, int64_t n, int64_t k, int dtype, void* stream);
 int b2l_moe_gemm_mma(void* c, const void* a, const void* w, const void* slot_weight_f32, const void* sorted_token_ids,
                      const void* expert_ids, const void* num_tokens_post_padded, int64_t em, int64_t num_valid_slots,
                      int top_k, int block_size, int64_t n, int64_t k, int64_t a_row_stride, int64_t c_row_stride,
-                     int act, int dtype, void* stream);
+                     int act, float limit, float alpha, int dtype, void* stream);
 /* Sigmoid scores + selection bias + group-limited top-k (csrc/moe_routing.cu); the router product is done inside
  * unless logits_f32 [tokens, experts] (nullable) brings it:
  * z = router_w . x in fp32, s = sigmoid(z), choice = s + bias (nullable); `groups` equal runs of neighbouring experts,
  * group score = sum of its two largest choice scores, only the `keep` best groups are eligible; the top_k largest
  * choice scores win; weights_f32 [tokens, top_k] = s of the winners / (their sum + 1e-20), or with renormalize 0 the
- * winners' s themselves; ids_i32 [tokens, top_k]. */
+ * winners' s themselves; ids_i32 [tokens, top_k].  softmax: s is the softmax over all experts; scale multiplies the
+ * weights. */
 int b2l_moe_route_sigmoid_groups(void* weights_f32, void* ids_i32, const void* x, int64_t x_row_stride,
                                  const void* router_w, const void* bias, const void* logits_f32, int64_t tokens,
                                  int num_experts, int64_t k, int top_k, int groups, int keep, int renormalize,
-                                 int dtype, void* stream);
+                                 int softmax, float scale, int dtype, void* stream);
 /* y_f32[m, n] = x[m, k] . w[n, k]^T: 16-bit operands on the tensor cores, the fp32 sums stored unrounded (router
  * logits); operands as b2l_rows_gemm_mma_ok asks. */
 int b2l_linear_f32out_mma(void* y_f32, const void* x, const void* w, int64_t m, int64_t n, int64_t k,
@@ -327,23 +330,24 @@ int b2l_linear_f32out_mma(void* y_f32, const void* x, const void* w, int64_t m, 
 int b2l_rope_table(void* cos_sin_f32, const void* pos_i32, int64_t tokens, int rot_dims, float rot_base, void* stream);
 /* Latent attention, per token of the fused down-projection row [a: q_rank | b: kv_rank | r: rot_dim | ...]:
  * a <- rmsnorm(a) * q_norm_weight in place; pool row kv_rows[t] = [rmsnorm(b) * kv_norm_weight | r with its first
- * rot_dims entries rotated by the token's row of cos_sin_f32 (entry i pairs with i + rot_dims / 2)]. */
+ * rot_dims entries rotated by the token's row of cos_sin_f32 (pairing 1: entry i pairs with i + rot_dims / 2, 0:
+ * neighbours 2i, 2i + 1)]. */
 int b2l_latent_prepare(void* proj, int64_t proj_row_stride, void* pool, int64_t pool_row_stride,
                        const void* kv_rows_i32, const void* cos_sin_f32, const void* q_norm_weight,
                        const void* kv_norm_weight, int64_t tokens, int q_rank, int kv_rank, int rot_dim, int rot_dims,
-                       float eps, int dtype, void* stream);
+                       int pairing, float eps, int dtype, void* stream);
 /* dst[t, h, :width] = src[t, h, :width], the first rot_dims entries rotated by the token's row of cos_sin_f32. */
 int b2l_rope_heads(void* dst, int64_t dst_row_stride, int dst_head_stride, const void* src, int64_t src_row_stride,
                    int src_head_stride, const void* cos_sin_f32, int64_t tokens, int heads, int width, int rot_dims,
-                   int dtype, void* stream);
+                   int pairing, int dtype, void* stream);
 
-/* Short causal convolution per channel + SiLU (activation 1; 0 = none) over a ragged step, and the slot's tail (last
- * taps-1 inputs) update.
+/* Short causal convolution per channel (bias nullable) + SiLU (activation 1; 0 = none) over a ragged step (residual 1: the
+ * input itself is added first), and the slot's tail (last taps-1 inputs) update, one launch.
  * in: [tokens, >= channels] with row stride; weight [channels, taps] (last column = current token); tail
  * [slots, taps - 1, channels] in dtype. */
 int b2l_causal_conv_silu(void* out, const void* in, int64_t in_row_stride, const void* weight, const void* bias,
                          void* tail, const void* seq_start, const void* seq_ctx, const void* seq_slot, int64_t num_seqs,
-                         int64_t tokens, int channels, int taps, int activation, int dtype, void* stream);
+                         int64_t tokens, int channels, int taps, int activation, int residual, int dtype, void* stream);
 /* Scalar-decay state-space recurrence (csrc/ssm_scan.cu).  xbc rows = [x: heads*head_dim | B: groups*state | C: ...];
  * state_f32 [slots, heads, state, head_dim] fp32; y_f32 [tokens, heads*head_dim] fp32.  fixed_decay_f32 [heads]
  * (nullable): decayed linear attention S <- decay_h S + B x^T, y = S^T C with dt = 1 and no skip term (dt_raw, dt_bias,
@@ -375,7 +379,9 @@ int b2l_attn_prepare(void* qkv, int64_t qkv_row_stride, void* kv_pool, int64_t k
 /* Soft-capped attention with an optional per-head sink over the pool (csrc/attention_sink.cu).  num_splits == 0: tiled
  * mode for sequences of up to max_q_len new tokens; num_splits > 0: every listed sequence brings one token, its keys
  * (from the first one it sees) are cut into num_splits ranges of split_keys and merged (workspace:
- * b2l_sink_attention_workspace_bytes).  window > 0: token p sees keys p - window + 1 .. p only; block > 0 (window <= 0):
+ * b2l_sink_attention_workspace_bytes).  window > 0: token p sees keys p - window + 1 .. p only, and with keep_first > 0
+ * also the sequence's first keep_first positions; gate (nullable) [tokens, >= heads]: head h's output times
+ * sigmoid(gate[t, h]); block > 0 (window <= 0):
  * token p sees keys floor(p / block) * block .. p only.  v_col0 < 0: a pool
  * row is [keys | values]; v_col0 >= 0: the values start at that column (0: they are the keys' leading columns).
  * v_blocks > 1 (num_splits > 0 only): v_blocks neighbouring blocks of v_head_dim value columns in one call, each as
@@ -385,8 +391,9 @@ int b2l_sink_attention(void* out, int64_t out_row_stride, const void* q, int64_t
                        int64_t kv_row_stride, const void* table_i32, int64_t table_row_stride, const void* seq_start,
                        const void* seq_ctx, const void* seq_slot, const void* seq_list, int64_t num_seqs,
                        int max_q_len, const void* sink, int heads, int kv_heads, int head_dim, int v_head_dim,
-                       float scale, float softcap, int window, int block, int v_col0, int v_head_stride,
-                       int v_blocks, int num_splits, int split_keys, void* workspace, int64_t workspace_bytes, int dtype,
+                       float scale, float softcap, int window, int keep_first, int block, int v_col0,
+                       int v_head_stride, int v_blocks, const void* gate, int64_t gate_row_stride, int num_splits,
+                       int split_keys, void* workspace, int64_t workspace_bytes, int dtype,
                        void* stream);
 /* One new token per listed sequence, the heads' softmax weights mixed across heads before the values:
  * p'_h(j) = sum_g mix[h, g] p_g(j), out_h = sum_j p'_h(j) v_kv(h)(j).  mix [heads, heads] has q's element type.  max_keys
@@ -447,29 +454,63 @@ int b2l_gated_linear_scan(void* y_f32, void* state_f32, const void* q, int64_t q
                           const void* seq_start, const void* seq_ctx, const void* seq_slot, int64_t num_seqs, int heads,
                           int qk_heads, int dim, int vdim, float q_scale, float unit_eps, int mode, int dtype,
                           void* stream);
-/* out[t, h, :] = unit_rms(y_f32[t, h, :]) * weight[vdim] * silu(gate[t, h, :]) (gate nullable: no gate). */
+/* out[t, h, :] = unit_rms(y_f32[t, h, :]) * weight[vdim] * silu(gate[t, h, :]) (gate nullable: no gate; sigmoid_gate 1:
+ * sigmoid instead of silu; head_weight 1: weight is [heads * vdim]). */
 int b2l_head_norm_gate(void* out, const void* y_f32, const void* gate, int64_t gate_row_stride, const void* weight,
-                       int64_t rows, int heads, int vdim, float eps, int dtype, void* stream);
+                       int64_t rows, int heads, int vdim, float eps, int sigmoid_gate, int head_weight, int dtype,
+                       void* stream);
 /* out[t, h, :] = sum_g mix[h, g] * wide[t, g, kv(h), :] for wide [rows, calls, heads, per_call, vdim] (kv head c of
  * query head g lies at call c / per_call, part c % per_call): softmax weights mixed across heads, on the outputs. */
 int b2l_head_mix(void* out, const void* wide, int64_t wide_row_stride, const void* mix, int64_t rows, int heads,
                  int kv_heads, int per_call, int vdim, int dtype, void* stream);
 /* out[r, :] = silu(s_r * gate[r, :]) * (s_r * up[r, :]) * sigmoid(z[r]); in_scale_f32 [rows] and z (one value per row,
- * row stride given) are nullable. */
+ * row stride given) are nullable.  form 1: the clamped unit g' sigmoid(alpha g') (u' + 1) instead of silu(g) u. */
 int b2l_swiglu_scaled(void* out, int64_t out_row_stride, const void* gate, int64_t gate_row_stride, const void* up,
                       int64_t up_row_stride, const void* in_scale_f32, const void* z, int64_t z_row_stride, int64_t rows,
-                      int64_t n, int dtype, void* stream);
+                      int64_t n, int form, float limit, float alpha, int dtype, void* stream);
+
+/* Matrix memory with exponential gates (csrc/mlstm.cu); state_f32 [slots, heads, b2l_mlstm_head_floats] = per head
+ * [S: dim x vdim | n: dim | m | pad], advanced in place; y_f32 [tokens, heads * vdim].  With i = cap tanh((zi + bi) / cap),
+ * f = logsigmoid(cap tanh((zf + bf) / cap)) per head (gate_cap <= 0: no bound), m' = max(f + m, i):
+ * S <- e^(f + m - m') S + e^(i - m') k v^T, n likewise, y = S^T q / (max(|n . q|, e^(-m')) + 1e-6), q times q_scale.
+ * seq_list (nullable): the sequences of this call.  chunked 0: token by token (dim <= 256); 1: 64-token chunks on the
+ * tensor cores (16-bit dtypes, dim <= 128).  tickets_i32: num_seqs * heads zeroed counters, left zeroed. */
+int64_t b2l_mlstm_head_floats(int dim, int vdim);
+int b2l_mlstm(void* y_f32, void* state_f32, const void* q, int64_t q_row_stride, const void* k, int64_t k_row_stride,
+              const void* v, int64_t v_row_stride, const void* zi, int64_t zi_row_stride, const void* zf,
+              int64_t zf_row_stride, const void* bi, const void* bf, const void* seq_start, const void* seq_ctx,
+              const void* seq_slot, const void* seq_list, int64_t num_seqs, int heads, int dim, int vdim, float q_scale,
+              float gate_cap, void* tickets_i32, int64_t num_tickets, int chunked, int dtype, void* stream);
+
+/* Residual streams x [tokens, streams, n] fp32 (csrc/hyper_stream.cu), up to 8 streams.  A read: u = sum_s in[s] x_s,
+ * h = unit_rms(u) * weight in dtype; with taps > 0 (steps in which every token is a sequence of its own) also
+ * hc = h + causal convolution of h (conv_w [n, taps], tail [slots, taps - 1, n] advanced).
+ * stream_embed: all streams = unit_rms(embed[token]) * embed_weight, then a read.
+ * stream_mix: x_t <- sum_s mix[s, t] x_s + out[t] y', then a read; y' = (sum of the token's `terms` rows of y + y2
+ * (nullable)) * sigmoid(z + z_bias) (z nullable: no gate); coef_f32 = [out: streams | mix: streams x streams].  rows_i32
+ * (nullable): only these tokens (`tokens` of them), h compact, the streams are not written. */
+int b2l_stream_embed(void* streams_f32, const void* tokens_i32, const void* embed, const void* embed_weight,
+                     int64_t vocab, const void* in_f32, const void* weight, void* h, const void* conv_w, void* tail,
+                     void* hc, const void* seq_ctx, const void* seq_slot, int taps, int64_t tokens, int streams,
+                     int64_t n, float eps, int dtype, void* stream);
+int b2l_stream_mix(void* streams_f32, const void* y, int64_t y_row_stride, int terms, const void* y2,
+                   int64_t y2_row_stride, const void* z, int64_t z_row_stride, const void* z_bias, const void* coef_f32,
+                   const void* in_f32, const void* weight, void* h, const void* rows_i32, const void* conv_w, void* tail,
+                   void* hc, const void* seq_ctx, const void* seq_slot, int taps, int64_t tokens, int streams, int64_t n,
+                   float eps, int dtype, void* stream);
 
 /* Rotary table from given per-pair frequencies (csrc/rotary_heads.cu): cos_sin_f32[t] = magnitude * [cos(pos f_i) |
  * sin(pos f_i)], fp64 frequencies and angles.  head_norm_rope_prepare: per token of a fused [q | k | v] row, per-head RMS norm of q and
  * k with one [head_dim] weight each (nullable), rotation of the first rot_dims entries (pairing 0: neighbours 2i, 2i+1;
- * 1: i and i + rot_dims / 2), q in place, k and v into pool row kv_rows[t]. */
+ * 1: i and i + rot_dims / 2), q in place, k and v into pool row kv_rows[t]; v_norm: every v head is divided by its root
+ * mean square first; kv_heads 0: q alone (kv_pool, kv_rows_i32 unused). */
 int b2l_rope_table_freqs(void* cos_sin_f32, const void* pos_i32, const void* freqs_f64, int64_t tokens, int rot_dims,
                          float magnitude, void* stream);
 int b2l_head_norm_rope_prepare(void* qkv, int64_t qkv_row_stride, void* kv_pool, int64_t kv_row_stride,
                                const void* kv_rows_i32, const void* cos_sin_f32, const void* q_norm_weight,
                                const void* k_norm_weight, int64_t tokens, int heads, int kv_heads, int head_dim,
-                               int v_head_dim, int rot_dims, int pairing, float eps, int dtype, void* stream);
+                               int v_head_dim, int rot_dims, int pairing, int v_norm, float eps, int dtype,
+                               void* stream);
 
 #ifdef __cplusplus
 }

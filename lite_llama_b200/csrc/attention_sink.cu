@@ -6,6 +6,8 @@
 // how a latent cache [latent | rotated key part] is read by queries that were multiplied into the latent space).
 // A sliding window (`window` > 0) limits token p to the keys p - window + 1 .. p; a block-diagonal mask (`block` > 0)
 // to the keys of its own run of `block` positions, floor(p / block) * block .. p (runs are counted from position 0).
+// `keep` > 0 (with a window): the sequence's first `keep` positions stay visible to every later token.  `gate`
+// (nullable, [tokens, >= heads]): head h's output is multiplied by sigmoid(gate[t, h]).
 //
 //   attn_prepare   per token: whole-row RMS norm of q and of k (one statistic over ALL heads, plain weight),
 //                  position-dependent query gain, value mixing with an earlier layer's values, K|V cache write
@@ -48,6 +50,8 @@ struct AttnArgs {
   int head_rows;               // tensor-core kernel, one new token per sequence: the tile's rows are the query HEADS of
                                // one kv head (not tokens), blockIdx.x is a key range, results go to `part`
   float scale, softcap;
+  int keep;                    // window only: key positions below `keep` are visible to every later token
+  const void* gate; int64_t gate_stride;      // per-head logistic output gate (nullable)
 };
 
 // first key position the token at `pos` sees (may be negative under a window: callers clamp where they index);
@@ -55,6 +59,20 @@ struct AttnArgs {
 __device__ __forceinline__ int first_visible(const AttnArgs& a, int pos) {
   return a.window > 0 ? pos - a.window + 1 : (a.block > 0 ? pos - pos % a.block : 0);
 }
+
+// One new token at position `ctx` sees the kept positions in front of its window and the window itself: two runs of
+// positions.  The single-token kernels walk ONE axis [lo, ctx]: coordinates from the window's first key on are key
+// positions, the `kept` coordinates in front of it are the kept positions.
+struct SeenAxis {
+  int win_lo, lo;              // window's first key; first coordinate (win_lo - kept)
+  __device__ __forceinline__ SeenAxis(const AttnArgs& a, int ctx) {
+    win_lo = max(0, first_visible(a, ctx));
+    lo = win_lo - min(a.keep, win_lo);
+  }
+  __device__ __forceinline__ int key(int c) const { return c < win_lo ? c - lo : c; }
+};
+
+__device__ __forceinline__ float gate_of(float z) { return 1.0f / (1.0f + expf(-z)); }
 
 // ---- tiled mode on the CUDA cores (fp32 activations, or head sizes the tensor-core tiles do not take) ------------
 template <typename T, int DVJ>
@@ -76,6 +94,7 @@ __global__ void __launch_bounds__(kWarps * 32) sink_attention_kernel(AttnArgs a)
   const int t_count = min(a.BQ, qlen - t0);
   const int key_hi = ctx + t0 + t_count;                // exclusive
   const int key_lo = max(0, first_visible(a, ctx + t0));                      // first key the tile's first token sees
+  const int keep_hi = min(a.keep, key_hi);               // kept positions in front of the window come first
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const T* q = (const T*)a.q;
   const T* kv = (const T*)a.kv;
@@ -98,16 +117,19 @@ __global__ void __launch_bounds__(kWarps * 32) sink_attention_kernel(AttnArgs a)
   }
   const int* trow = a.table + slot * a.table_stride;
   const float inv_cap = a.softcap > 0.f ? 1.0f / a.softcap : 0.f;
-  for (int k0 = key_lo; k0 < key_hi; k0 += kKeys) {
+  for (int k0 = (keep_hi > 0 && key_lo > 0) ? 0 : key_lo; k0 < key_hi;
+       k0 = (k0 + kKeys >= keep_hi && k0 + kKeys < key_lo) ? key_lo : k0 + kKeys) {
     __syncthreads();
     const int nk = min(kKeys, key_hi - k0);
     for (int i = tid; i < kKeys * D; i += blockDim.x) {
       const int j = i / D, d = i - j * D;
-      ks[j * (D + 1) + d] = j < nk ? to_f32(kv[(int64_t)trow[k0 + j] * a.kv_stride + g * D + d]) : 0.f;
+      const bool in = j < nk && (k0 + j >= key_lo || k0 + j < keep_hi);       // positions no row sees may have no row
+      ks[j * (D + 1) + d] = in ? to_f32(kv[(int64_t)trow[k0 + j] * a.kv_stride + g * D + d]) : 0.f;
     }
     for (int i = tid; i < kKeys * Dv; i += blockDim.x) {
       const int j = i / Dv, d = i - j * Dv;
-      vs[i] = j < nk ? to_f32(kv[(int64_t)trow[k0 + j] * a.kv_stride + a.v_col0 + g * a.v_hstride + d]) : 0.f;
+      const bool in = j < nk && (k0 + j >= key_lo || k0 + j < keep_hi);
+      vs[i] = in ? to_f32(kv[(int64_t)trow[k0 + j] * a.kv_stride + a.v_col0 + g * a.v_hstride + d]) : 0.f;
     }
     __syncthreads();
     float sc[kRowsPerWarp];
@@ -124,12 +146,13 @@ __global__ void __launch_bounds__(kWarps * 32) sink_attention_kernel(AttnArgs a)
     for (int i = 0; i < kRowsPerWarp; ++i) {
       if (row_pos[i] < k0) continue;              // warp-uniform: nothing visible in this tile (or unused row)
       const int row_lo = first_visible(a, row_pos[i]);
-      if (row_lo >= k0 + nk) continue;            // warp-uniform: the row's window starts after this tile
+      if (row_lo >= k0 + nk && k0 >= keep_hi) continue;      // warp-uniform: the row's window starts after this tile
       float sv = sc[i] * a.scale;
       if (a.softcap > 0.f) sv = a.softcap * tanhf(sv * inv_cap);
-      const bool ok = lane < nk && k0 + lane <= row_pos[i] && k0 + lane >= row_lo;
+      const bool ok = lane < nk && k0 + lane <= row_pos[i] && (k0 + lane >= row_lo || k0 + lane < keep_hi);
       sv = ok ? sv : -INFINITY;
       const float mt = warp_reduce_max(sv);
+      if (mt == -INFINITY) continue;               // warp-uniform: the row sees no key of this tile
       const float mn = fmaxf(m[i], mt);
       const float corr = expf(m[i] - mn);          // exp(-inf) = 0 on the first tile
       const float p = ok ? expf(sv - mn) : 0.f;
@@ -159,7 +182,8 @@ __global__ void __launch_bounds__(kWarps * 32) sink_attention_kernel(AttnArgs a)
         num = expf(m[i] - mf);
         den = l[i] * num + expf(sk - mf);
       }
-      const float inv = num / den;
+      float inv = num / den;
+      if (a.gate) inv *= gate_of(to_f32(((const T*)a.gate)[(int64_t)(start + t0 + tl) * a.gate_stride + h]));
       T* o = (T*)a.out + (int64_t)(start + t0 + tl) * a.out_stride + h * Dv;
 #pragma unroll
       for (int j = 0; j < DVJ; ++j) {
@@ -218,8 +242,8 @@ __global__ void __launch_bounds__(128) sink_attention_mma_kernel(AttnArgs a) {
   const int t_count = hr ? min(kTileM, g * per + per - h_base) : min(kTileM, qlen - t0);       // live rows
   const int h = h_base;
   const int64_t slot = a.seq_slot[s];
-  const int win_lo = max(0, first_visible(a, ctx));                            // head rows: the token's first visible key
-  const int range_lo = hr ? win_lo + blockIdx.x * a.chunk : 0;
+  const SeenAxis axis(a, ctx);                                                  // head rows: what the one token sees
+  const int range_lo = hr ? axis.lo + blockIdx.x * a.chunk : 0;
   const int key_hi = hr ? min(range_lo + a.chunk, ctx + 1) : ctx + t0 + t_count;               // exclusive
   const bool ok0 = r0 < t_count, ok1 = r1 < t_count;
   const int pos0 = hr ? key_hi - 1 : ctx + t0 + r0, pos1 = hr ? key_hi - 1 : ctx + t0 + r1;     // last visible key of each row
@@ -228,6 +252,15 @@ __global__ void __launch_bounds__(128) sink_attention_mma_kernel(AttnArgs a) {
   // first key tile: the one that holds the first key of the tile's first row (tiles stay aligned to kTileN)
   const int k_first = hr ? range_lo / kTileN * kTileN : max(0, first_visible(a, ctx + t0)) / kTileN * kTileN;
   const int warp_first = hr ? range_lo : first_visible(a, ctx + t0 + warp * 16);                    // first key of the warp's rows
+  // token rows: kept positions in front of the window are tiles of their own; positions between them and the window
+  // are not read
+  const int keep_hi = hr ? 0 : min(a.keep, key_hi);
+  const int tile_lo = hr ? range_lo : max(0, first_visible(a, ctx + t0));
+  auto next_tile = [&](int k0) {
+    k0 += kTileN;
+    return (k0 >= keep_hi && k0 < k_first) ? k_first : k0;
+  };
+  auto row_of = [&](int k) { return (k < key_hi && (k >= tile_lo || k < keep_hi)) ? (hr ? axis.key(k) : k) : -1; };
   const T* q = (const T*)a.q;
   const T* kv = (const T*)a.kv;
   uint32_t qf[DP / 16][4];
@@ -264,12 +297,14 @@ __global__ void __launch_bounds__(128) sink_attention_mma_kernel(AttnArgs a) {
 #pragma unroll
     for (int j = 0; j < JK; ++j) {
       const int r = (tid + 128 * j) / (DP / 8);
-      rk[j] = k0 + r < key_hi ? trow[k0 + r] : -1;
+      const int k = row_of(k0 + r);
+      rk[j] = k >= 0 ? trow[k] : -1;
     }
 #pragma unroll
     for (int j = 0; j < JV; ++j) {
       const int r = (tid + 128 * j) / (DVP / 8);
-      rv[j] = k0 + r < key_hi ? trow[k0 + r] : -1;
+      const int k = row_of(k0 + r);
+      rv[j] = k >= 0 ? trow[k] : -1;
     }
 #pragma unroll
     for (int j = 0; j < JK; ++j) {
@@ -289,15 +324,17 @@ __global__ void __launch_bounds__(128) sink_attention_mma_kernel(AttnArgs a) {
     }
     cp_async_commit();
   };
-  if (k_first < key_hi) issue(k_first, 0);
-  for (int k0 = k_first, it = 0; k0 < key_hi; k0 += kTileN, ++it) {
-    const bool more = k0 + kTileN < key_hi;
-    if (more) issue(k0 + kTileN, (it + 1) & 1);                  // the next tile flies while this one is used
+  const int k_start = (keep_hi > 0 && k_first > 0) ? 0 : k_first;
+  if (k_start < key_hi) issue(k_start, 0);
+  for (int k0 = k_start, it = 0, kn; k0 < key_hi; k0 = kn, ++it) {
+    kn = next_tile(k0);
+    const bool more = kn < key_hi;
+    if (more) issue(kn, (it + 1) & 1);                           // the next tile flies while this one is used
     if (more) cp_async_wait<1>(); else cp_async_wait<0>();
     __syncthreads();                                             // tile `it` is complete and visible to every warp
     const uint32_t ks = smem_u32(smem_raw + (it & 1) * kStage), vs = ks + kTileN * KP;
     // the barrier at the END of the body keeps stage it & 1 intact until every warp is done with it
-    if (k0 > warp_last || k0 + kTileN <= warp_first) { __syncthreads(); continue; }
+    if (k0 > warp_last || (k0 + kTileN <= warp_first && k0 >= keep_hi)) { __syncthreads(); continue; }
     float sc[kTileN / 8][4];
 #pragma unroll
     for (int j = 0; j < kTileN / 8; ++j) sc[j][0] = sc[j][1] = sc[j][2] = sc[j][3] = 0.f;
@@ -324,7 +361,7 @@ __global__ void __launch_bounds__(128) sink_attention_mma_kernel(AttnArgs a) {
         const int lim = (e >> 1) ? pos1 : pos0, first = (e >> 1) ? lo1 : lo0;
         float v = sc[j][e] * a.scale;
         if (cap > 0.f) v = cap * tanh_fast(v * inv_cap);
-        v = (key <= lim && key >= first) ? v * kLog2e : -INFINITY;
+        v = (key <= lim && (key >= first || key < keep_hi)) ? v * kLog2e : -INFINITY;
         sc[j][e] = v;
         mx[e >> 1] = fmaxf(mx[e >> 1], v);
       }
@@ -409,6 +446,8 @@ __global__ void __launch_bounds__(128) sink_attention_mma_kernel(AttnArgs a) {
       den = l_run[r2] * num + fast_exp2(sk - mf);
     }
     inv[r2] = num / den;
+    if (a.gate && (r2 ? ok1 : ok0))
+      inv[r2] *= gate_of(to_f32(((const T*)a.gate)[(int64_t)(start + t0 + (r2 ? r1 : r0)) * a.gate_stride + h]));
   }
   T* ob = (T*)a.out + h * Dv;
   if (ok0) {
@@ -489,8 +528,8 @@ __global__ void __launch_bounds__(128) sink_attention_split_kernel(AttnArgs a) {
   const int g = by / hchunks, h_first = g * per + (by % hchunks) * kSplitRows;
   const int h_count = min(kSplitRows, g * per + per - h_first);
   const int v_col = a.v_col0 + vb * Dv + g * a.v_hstride;                    // first value column of this CTA
-  const int win_lo = max(0, first_visible(a, ctx));                          // the new token's first visible key
-  const int key_lo = win_lo + blockIdx.x * a.chunk, key_hi = min(key_lo + a.chunk, ctx + 1);
+  const SeenAxis axis(a, ctx);                                               // what the new token sees
+  const int key_lo = axis.lo + blockIdx.x * a.chunk, key_hi = min(key_lo + a.chunk, ctx + 1);
   const T* q = (const T*)a.q;
   const T* kv = (const T*)a.kv;
   const int Dq = (D + 3) / 4 * 4;
@@ -516,7 +555,7 @@ __global__ void __launch_bounds__(128) sink_attention_split_kernel(AttnArgs a) {
     if (vec_ok) {
       // lane j fetches key j's pool row once; the 16-byte copies run in batches of kStageBatch loads per lane that
       // are all in flight before the first shared-memory store
-      const int my_row = lane < nk ? trow[k0 + lane] : 0;
+      const int my_row = lane < nk ? trow[axis.key(k0 + lane)] : 0;
       auto stage_rows = [&](T* dst, int pitch, int col0, int vecs) {
         for (int base = 0; base < nk * vecs; base += 32 * kStageBatch) {
           uint4 raw[kStageBatch];
@@ -539,11 +578,11 @@ __global__ void __launch_bounds__(128) sink_attention_split_kernel(AttnArgs a) {
     } else {
       for (int i = lane; i < nk * D; i += 32) {
         const int j = i / D, d = i - j * D;
-        ks[j * Dp + d] = kv[(int64_t)trow[k0 + j] * a.kv_stride + g * D + d];
+        ks[j * Dp + d] = kv[(int64_t)trow[axis.key(k0 + j)] * a.kv_stride + g * D + d];
       }
       for (int i = lane; i < nk * Dv; i += 32) {
         const int j = i / Dv, d = i - j * Dv;
-        vs[j * Dvp + d] = kv[(int64_t)trow[k0 + j] * a.kv_stride + v_col + d];
+        vs[j * Dvp + d] = kv[(int64_t)trow[axis.key(k0 + j)] * a.kv_stride + v_col + d];
       }
     }
     __syncwarp();
@@ -672,7 +711,8 @@ __global__ void __launch_bounds__(64) sink_attention_merge_kernel(T* __restrict_
                                                                   const T* __restrict__ sink,
                                                                   const int* __restrict__ seq_start,
                                                                   const int* __restrict__ seq_list, int H, int Dv,
-                                                                  int nsplit, int sink_heads) {
+                                                                  int nsplit, int sink_heads,
+                                                                  const T* __restrict__ gate, int64_t gate_stride) {
   pdl_prologue();
   __shared__ float wsm[kMergeCached];
   __shared__ float red[2];
@@ -699,13 +739,15 @@ __global__ void __launch_bounds__(64) sink_attention_merge_kernel(T* __restrict_
   den = red[0] + red[1];
   if (sink) den += expf(to_f32(sink[h % sink_heads]) - mf);
   T* o = out + (int64_t)seq_start[s] * out_stride + h * Dv;
+  float num = 1.0f;
+  if (gate) num = gate_of(to_f32(gate[(int64_t)seq_start[s] * gate_stride + h % sink_heads]));
   for (int d = tid; d < Dv; d += 64) {
     float v = 0.f;
     for (int i = 0; i < nsplit; ++i) {
       const float w = i < kMergeCached ? wsm[i] : expf(p[i * (Dv + 2)] - mf);
       v = fmaf(p[i * (Dv + 2) + 2 + d], w, v);
     }
-    o[d] = from_f32<T>(v / den);
+    o[d] = from_f32<T>(gate ? v / den * num : v / den);
   }
 }
 
@@ -1089,8 +1131,9 @@ extern "C" int64_t b2l_sink_attention_workspace_bytes(int64_t num_seqs, int head
 
 /* num_splits == 0: tiled mode over `max_q_len`-token sequences; > 0: split mode, every listed sequence brings ONE token
  * and `split_keys` keys go to each of the num_splits ranges, counted from the token's first visible key
- * (num_splits * split_keys >= the most keys any listed token sees: context + 1, or the window if that is smaller).
- * window <= 0: no sliding window; block > 0 (window <= 0): block-diagonal mask; v_col0 < 0: the values follow the keys in a pool row (column kv_heads * head_dim);
+ * (num_splits * split_keys >= the most keys any listed token sees: context + 1, or window + keep_first if that is
+ * smaller).  window <= 0: no sliding window; keep_first (with a window): the first positions that stay visible;
+ * gate (nullable) [tokens, >= heads]: head h's output times sigmoid(gate[t, h]); block > 0 (window <= 0): block-diagonal mask; v_col0 < 0: the values follow the keys in a pool row (column kv_heads * head_dim);
  * v_head_stride < 0: kv head g's values start g * v_head_dim columns after v_col0 (0: all kv heads read the same columns).
  * v_blocks > 1 (split mode): block c of v_head_dim value columns starts c * v_head_dim columns further and is one more
  * set of `heads` results, out [v_blocks][heads][v_head_dim] per token, in the same two launches (workspace for
@@ -1100,8 +1143,9 @@ extern "C" int b2l_sink_attention(void* out, int64_t out_row_stride, const void*
                                   int64_t table_row_stride, const void* seq_start, const void* seq_ctx,
                                   const void* seq_slot, const void* seq_list, int64_t num_seqs, int max_q_len,
                                   const void* sink, int heads, int kv_heads, int head_dim, int v_head_dim, float scale,
-                                  float softcap, int window, int block, int v_col0, int v_head_stride, int v_blocks,
-                                  int num_splits, int split_keys, void* workspace, int64_t workspace_bytes, int dtype, void* stream) {
+                                  float softcap, int window, int keep_first, int block, int v_col0, int v_head_stride,
+                                  int v_blocks, const void* gate, int64_t gate_row_stride, int num_splits,
+                                  int split_keys, void* workspace, int64_t workspace_bytes, int dtype, void* stream) {
   B2L_REQUIRE(out && q && kv_pool && table_i32 && seq_start && seq_ctx && seq_slot, "sink_attention: null pointer");
   B2L_REQUIRE(heads > 0 && kv_heads > 0 && heads % kv_heads == 0, "sink_attention: %d heads must be a multiple of num_kv_heads %d",
               heads, kv_heads);
@@ -1121,6 +1165,8 @@ extern "C" int b2l_sink_attention(void* out, int64_t out_row_stride, const void*
   a.nsplit = num_splits; a.chunk = split_keys; a.scale = scale; a.softcap = softcap;
   a.window = window > 0 ? window : 0;
   a.block = (window <= 0 && block > 0) ? block : 0;
+  a.keep = (window > 0 && keep_first > 0) ? keep_first : 0;
+  a.gate = gate; a.gate_stride = gate_row_stride;
   a.v_col0 = v_col0 >= 0 ? v_col0 : kv_heads * head_dim;
   a.v_hstride = v_head_stride >= 0 ? v_head_stride : v_head_dim;
   a.head_rows = 0;
@@ -1147,7 +1193,8 @@ extern "C" int b2l_sink_attention(void* out, int64_t out_row_stride, const void*
     B2L_DISPATCH_FLOAT(dtype, "sink_attention", {
       b2l_launch(sink_attention_merge_kernel<T>, dim3((unsigned)(heads * a.v_blocks), (unsigned)num_seqs), dim3(64),
                  (size_t)0, st, (T*)out, out_row_stride, (const float*)workspace, (const T*)sink,
-                 (const int*)seq_start, (const int*)seq_list, heads * a.v_blocks, v_head_dim, num_splits, heads);
+                 (const int*)seq_start, (const int*)seq_list, heads * a.v_blocks, v_head_dim, num_splits, heads,
+                 (const T*)gate, gate_row_stride);
     });
     B2L_LAUNCH_CHECK();
     return B2L_OK;

@@ -20,15 +20,16 @@
 // to back.  A sequence without cached tokens starts from zero and never
 // reads its slot; every sequence writes its slot at the end of the step.
 //
-//   head_norm_gate   out[t, h, :] = unit_rms(y[t, h, :]) * w * (silu(gate[t, h, :]) or 1): the per-head output norm
-//                    (weight [V] shared by the heads) with an optional SiLU gate AFTER the norm
+//   head_norm_gate   out[t, h, :] = unit_rms(y[t, h, :]) * w * (silu(gate[t, h, :]), sigmoid of it, or 1): the per-head
+//                    output norm (weight [V] shared by the heads, or [H * V]) with an optional gate AFTER the norm
 //   head_mix         out[t, h, :] = sum_g M[h, g] * wide[t, g, kv(h), :]: attention weights mixed ACROSS heads after
 //                    the softmax, done on per-head outputs -- head g's weights were applied to every kv head's values
 //                    (sum_j (sum_g M[h,g] p_g(j)) v(j) = sum_g M[h,g] (sum_j p_g(j) v(j)))
 //   swiglu_scaled    out[r, :] = silu(s_r * gate) * (s_r * up) * sigmoid(z_r): a gated activation whose INPUT carries
 //                    a per-row fp32 factor (an expert weight on the expert's input: W (s x) = s (W x)) and whose output
-//                    a per-row logistic gate (both optional)
+//                    a per-row logistic gate (both optional); the unit may be the clamped form of gated_unit.cuh instead
 #include "common.cuh"
+#include "gated_unit.cuh"
 #include "rowvec.cuh"
 
 namespace {
@@ -270,13 +271,14 @@ __global__ void __launch_bounds__(kScanThreads, 2) gated_linear_scan_kernel(GlaA
 template <typename T>
 __global__ void __launch_bounds__(128) head_norm_gate_kernel(T* __restrict__ out, const float* __restrict__ y,
                                                              const T* __restrict__ gate, int64_t gs,
-                                                             const T* __restrict__ w, int heads, int V, float eps,
-                                                             int vec) {
+                                                             const T* __restrict__ wt, int heads, int V, float eps,
+                                                             int vec, int sigmoid_gate, int head_weight) {
   pdl_prologue();
   const int64_t t = blockIdx.x;
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
   for (int h = warp; h < heads; h += nw) {
     const float* yr = y + (t * heads + h) * (int64_t)V;
+    const T* w = wt + (head_weight ? (int64_t)h * V : 0);
     float ss = 0.f;
     if (vec) {                                       // 4 elements per access
       for (int i = lane * 4; i < V; i += 128) {
@@ -295,7 +297,7 @@ __global__ void __launch_bounds__(128) head_norm_gate_kernel(T* __restrict__ out
         if (gate) {
           row_load4(gate + t * gs + (int64_t)h * V + i, g);
 #pragma unroll
-          for (int c = 0; c < 4; ++c) v[c] *= gla_silu(g[c]);
+          for (int c = 0; c < 4; ++c) v[c] *= sigmoid_gate ? gla_sigmoid(g[c]) : gla_silu(g[c]);
         }
         row_store4(out + (t * heads + h) * (int64_t)V + i, v);
       }
@@ -305,7 +307,10 @@ __global__ void __launch_bounds__(128) head_norm_gate_kernel(T* __restrict__ out
     const float rstd = 1.0f / sqrtf(warp_reduce_sum(ss) / (float)V + eps);
     for (int i = lane; i < V; i += 32) {
       float v = yr[i] * rstd * to_f32(w[i]);
-      if (gate) v *= gla_silu(to_f32(gate[t * gs + (int64_t)h * V + i]));
+      if (gate) {
+        const float g = to_f32(gate[t * gs + (int64_t)h * V + i]);
+        v *= sigmoid_gate ? gla_sigmoid(g) : gla_silu(g);
+      }
       out[(t * heads + h) * (int64_t)V + i] = from_f32<T>(v);
     }
   }
@@ -395,7 +400,8 @@ __global__ void head_mix_group_kernel(T* __restrict__ out, const T* __restrict__
 template <typename T>
 __global__ void swiglu_scaled_vec_kernel(T* __restrict__ out, int64_t os, const T* __restrict__ gate, int64_t gs,
                                          const T* __restrict__ up, int64_t us, const float* __restrict__ in_scale,
-                                         const T* __restrict__ z, int64_t zs, int64_t n4, int64_t total4) {
+                                         const T* __restrict__ z, int64_t zs, int64_t n4, int64_t total4,
+                                         GatedUnit unit) {
   pdl_prologue();
   for (int64_t idx = blockIdx.x * (int64_t)blockDim.x + threadIdx.x; idx < total4; idx += (int64_t)gridDim.x * blockDim.x) {
     const int64_t r = idx / n4, i = (idx - r * n4) * 4;
@@ -405,7 +411,7 @@ __global__ void swiglu_scaled_vec_kernel(T* __restrict__ out, int64_t os, const 
     row_load4(gate + r * gs + i, g);
     row_load4(up + r * us + i, u);
 #pragma unroll
-    for (int e = 0; e < 4; ++e) g[e] = gla_silu(s * g[e]) * (s * u[e]) * zo;
+    for (int e = 0; e < 4; ++e) g[e] = unit(s * g[e], s * u[e]) * zo;
     row_store4(out + r * os + i, g);
   }
 }
@@ -413,14 +419,14 @@ __global__ void swiglu_scaled_vec_kernel(T* __restrict__ out, int64_t os, const 
 template <typename T>
 __global__ void swiglu_scaled_kernel(T* __restrict__ out, int64_t os, const T* __restrict__ gate, int64_t gs,
                                      const T* __restrict__ up, int64_t us, const float* __restrict__ in_scale,
-                                     const T* __restrict__ z, int64_t zs, int64_t n, int64_t total) {
+                                     const T* __restrict__ z, int64_t zs, int64_t n, int64_t total, GatedUnit unit) {
   pdl_prologue();
   for (int64_t idx = blockIdx.x * (int64_t)blockDim.x + threadIdx.x; idx < total; idx += (int64_t)gridDim.x * blockDim.x) {
     const int64_t r = idx / n, i = idx - r * n;
     const float s = in_scale ? in_scale[r] : 1.0f;
     const float g = s * to_f32(gate[r * gs + i]), u = s * to_f32(up[r * us + i]);
     const float zo = z ? gla_sigmoid(to_f32(z[r * zs])) : 1.0f;
-    out[r * os + i] = from_f32<T>(gla_silu(g) * u * zo);
+    out[r * os + i] = from_f32<T>(unit(g, u) * zo);
   }
 }
 
@@ -487,8 +493,8 @@ extern "C" int b2l_gated_linear_scan(void* y_f32, void* state_f32, const void* q
 }
 
 extern "C" int b2l_head_norm_gate(void* out, const void* y_f32, const void* gate, int64_t gate_row_stride,
-                                  const void* weight, int64_t rows, int heads, int vdim, float eps, int dtype,
-                                  void* stream) {
+                                  const void* weight, int64_t rows, int heads, int vdim, float eps, int sigmoid_gate,
+                                  int head_weight, int dtype, void* stream) {
   B2L_REQUIRE(out && y_f32 && weight, "head_norm_gate: null pointer");
   B2L_REQUIRE(heads > 0 && vdim > 0, "head_norm_gate: bad shape");
   if (rows <= 0) return B2L_OK;
@@ -498,7 +504,7 @@ extern "C" int b2l_head_norm_gate(void* out, const void* y_f32, const void* gate
     b2l_launch(head_norm_gate_kernel<T>, dim3((unsigned)rows), dim3(threads), (size_t)0, st, (T*)out, (const float*)y_f32,
                (const T*)gate, gate_row_stride, (const T*)weight, heads, vdim, eps,
                (int)(vdim % 4 == 0 && gate_row_stride % 4 == 0 && row_aligned4<T>(out) && row_aligned4<T>(gate) &&
-                     row_aligned4<T>(weight) && (uintptr_t)y_f32 % 16 == 0));
+                     row_aligned4<T>(weight) && (uintptr_t)y_f32 % 16 == 0), sigmoid_gate, head_weight);
   });
   B2L_LAUNCH_CHECK();
   return B2L_OK;
@@ -541,9 +547,11 @@ extern "C" int b2l_head_mix(void* out, const void* wide, int64_t wide_row_stride
 
 extern "C" int b2l_swiglu_scaled(void* out, int64_t out_row_stride, const void* gate, int64_t gate_row_stride,
                                  const void* up, int64_t up_row_stride, const void* in_scale_f32, const void* z,
-                                 int64_t z_row_stride, int64_t rows, int64_t n, int dtype, void* stream) {
+                                 int64_t z_row_stride, int64_t rows, int64_t n, int form, float limit, float alpha,
+                                 int dtype, void* stream) {
   B2L_REQUIRE(out && gate && up, "swiglu_scaled: null pointer");
-  B2L_REQUIRE(n > 0, "swiglu_scaled: bad shape");
+  B2L_REQUIRE(n > 0 && (form == kUnitSilu || form == kUnitClamped), "swiglu_scaled: bad shape or form %d", form);
+  const GatedUnit unit{form, limit, alpha};
   if (rows <= 0) return B2L_OK;
   cudaStream_t st = (cudaStream_t)stream;
   const int64_t total = rows * n;
@@ -553,12 +561,12 @@ extern "C" int b2l_swiglu_scaled(void* out, int64_t out_row_stride, const void* 
       const unsigned grid = (unsigned)(cdiv64(total / 4, 256) < 148 * 32 ? cdiv64(total / 4, 256) : 148 * 32);
       b2l_launch(swiglu_scaled_vec_kernel<T>, dim3(grid), dim3(256), (size_t)0, st, (T*)out, out_row_stride,
                  (const T*)gate, gate_row_stride, (const T*)up, up_row_stride, (const float*)in_scale_f32, (const T*)z,
-                 z_row_stride, n / 4, total / 4);
+                 z_row_stride, n / 4, total / 4, unit);
     } else {
       const unsigned grid = (unsigned)(cdiv64(total, 256) < 148 * 16 ? cdiv64(total, 256) : 148 * 16);
       b2l_launch(swiglu_scaled_kernel<T>, dim3(grid), dim3(256), (size_t)0, st, (T*)out, out_row_stride, (const T*)gate,
                  gate_row_stride, (const T*)up, up_row_stride, (const float*)in_scale_f32, (const T*)z, z_row_stride, n,
-                 total);
+                 total, unit);
     }
   });
   B2L_LAUNCH_CHECK();

@@ -1,6 +1,6 @@
 // Tensor-core (mma.sync m16n8k16, fp32 accumulators) versions of the two row-mapped products of csrc/gemm_simt.cu for
 // 16-bit activations:
-//   * per-head product   y[t, h, :] = W[h] . x[t, h, :]          (* sigmoid(gate[t, h]))
+//   * per-head product   y[t, h, :] = W[h] . x[t, h, :]          (* sigmoid(gate[t, h]), or one gate per element)
 //   * grouped product    c[s, :] = act(W[expert(s)] . a[s / top_k, :]) * slot_weight[s]     over expert-sorted slots
 // One kernel, two row maps: a CTA owns BM rows (16, 64 or 128) x 64 output columns of one head / one expert block, its
 // four warps hold 16-column slices (BM = 16), 16-row slices (BM = 64) or 32-row slices (BM = 128).  The rows' inputs are
@@ -10,6 +10,7 @@
 // a row's result does not depend on which other rows share its tile.  Needs k a multiple of 8 and 16-byte aligned rows
 // (the callers fall back to the CUDA-core kernels otherwise); W is [heads or experts, n, k] dense.
 #include "common.cuh"
+#include "gated_unit.cuh"
 
 namespace {
 
@@ -19,10 +20,11 @@ struct RowsArgs {
   const void* x; const void* w; void* y;
   int64_t n, k, xs, ys;
   // per-head map
-  int64_t m, xh, yh, gs; const void* gate;
+  int64_t m, xh, yh, gs; const void* gate; int gate_elements;
   // grouped map
   const float* slot_weight; const int* sorted_ids; const int* expert_ids; const int* num_post;
   int64_t num_valid; int top_k, act;
+  GatedUnit unit;              // act 2: columns 2i, 2i + 1 are gate i and up i, one output column i
   int out_f32;                 // per-head map only: y is fp32 (router logits: 16-bit operands, 32-bit sums kept as they are)
 };
 
@@ -69,7 +71,7 @@ __global__ void __launch_bounds__(128) rows_gemm_mma_kernel(RowsArgs a) {
       arow[tid] = ok ? (const T*)a.x + row * a.xs + h * a.xh : nullptr;
       const int64_t off = row * a.ys + h * a.yh;
       crow[tid] = ok ? (a.out_f32 ? (void*)((float*)a.y + off) : (void*)((T*)a.y + off)) : nullptr;
-      mult[tid] = (ok && a.gate) ? 1.0f / (1.0f + expf(-to_f32(((const T*)a.gate)[row * a.gs + h]))) : 1.0f;
+      mult[tid] = (ok && a.gate && !a.gate_elements) ? 1.0f / (1.0f + expf(-to_f32(((const T*)a.gate)[row * a.gs + h]))) : 1.0f;
     }
   }
   __syncthreads();
@@ -143,10 +145,20 @@ __global__ void __launch_bounds__(128) rows_gemm_mma_kernel(RowsArgs a) {
       continue;
     }
     T* dst = (T*)crow[r];
+    const T* ge = nullptr;                                     // the row's element gates of this head
+    if (!GROUPED && a.gate_elements) ge = (const T*)a.gate + ((int64_t)blockIdx.y * BM + r) * a.gs + blockIdx.z * a.n;
 #pragma unroll
     for (int j = 0; j < NT; ++j) {
       const int64_t col = n0 + wn * (NT * 8) + j * 8 + 2 * tq;
       float v0 = acc[mi][j][half * 2], v1 = acc[mi][j][half * 2 + 1];
+      if (!GROUPED && ge) {
+        if (col < a.n) v0 *= 1.0f / (1.0f + expf(-to_f32(ge[col])));
+        if (col + 1 < a.n) v1 *= 1.0f / (1.0f + expf(-to_f32(ge[col + 1])));
+      }
+      if (GROUPED && a.act == 2) {
+        if (col + 1 < a.n) dst[col >> 1] = from_f32<T>(a.unit(v0, v1) * g);
+        continue;
+      }
       if (GROUPED && a.act == 1) { v0 = gelu_erf_m(v0); v1 = gelu_erf_m(v1); }
       v0 *= g; v1 *= g;
       if (col + 1 < a.n && (((uintptr_t)(dst + col)) & 3) == 0) {
@@ -189,8 +201,8 @@ extern "C" int b2l_rows_gemm_mma_ok(const void* x, const void* w, int64_t k, int
 
 extern "C" int b2l_head_linear_mma(void* y, int64_t y_row_stride, int64_t y_head_stride, const void* x,
                                    int64_t x_row_stride, int64_t x_head_stride, const void* w, const void* gate,
-                                   int64_t gate_row_stride, int64_t m, int heads, int64_t n, int64_t k, int dtype,
-                                   void* stream) {
+                                   int64_t gate_row_stride, int gate_elements, int64_t m, int heads, int64_t n,
+                                   int64_t k, int dtype, void* stream) {
   B2L_REQUIRE(y && x && w, "head_linear_mma: null pointer");
   B2L_REQUIRE(m >= 0 && heads > 0 && heads <= 65535 && n > 0, "head_linear_mma: bad shape");
   B2L_REQUIRE(b2l_rows_gemm_mma_ok(x, w, k, x_row_stride, x_head_stride, dtype), "head_linear_mma: operands not aligned");
@@ -198,6 +210,7 @@ extern "C" int b2l_head_linear_mma(void* y, int64_t y_row_stride, int64_t y_head
   RowsArgs a = {};
   a.x = x; a.w = w; a.y = y; a.n = n; a.k = k; a.xs = x_row_stride; a.ys = y_row_stride;
   a.m = m; a.xh = x_head_stride; a.yh = y_head_stride; a.gs = gate_row_stride; a.gate = gate;
+  a.gate_elements = gate ? gate_elements : 0;
   const int bm = pick_rows(m, cdiv64(n, kBN) * heads);
   const dim3 grid((unsigned)cdiv64(n, kBN), (unsigned)cdiv64(m, bm), (unsigned)heads);
   cudaStream_t st = (cudaStream_t)stream;
@@ -212,9 +225,9 @@ extern "C" int b2l_moe_gemm_mma(void* c, const void* a_in, const void* w, const 
                                 const void* sorted_token_ids, const void* expert_ids,
                                 const void* num_tokens_post_padded, int64_t em, int64_t num_valid_slots, int top_k,
                                 int block_size, int64_t n, int64_t k, int64_t a_row_stride, int64_t c_row_stride,
-                                int act, int dtype, void* stream) {
+                                int act, float limit, float alpha, int dtype, void* stream) {
   B2L_REQUIRE(c && a_in && w && sorted_token_ids && expert_ids && num_tokens_post_padded, "moe_gemm_mma: null pointer");
-  B2L_REQUIRE(top_k >= 1 && n > 0 && em >= 0 && (act == 0 || act == 1) &&
+  B2L_REQUIRE(top_k >= 1 && n > 0 && em >= 0 && act >= 0 && act <= 2 && (act != 2 || n % 2 == 0) &&
                   (block_size == 16 || block_size == 64 || block_size == 128), "moe_gemm_mma: bad shape");
   B2L_REQUIRE(b2l_rows_gemm_mma_ok(a_in, w, k, a_row_stride, 0, dtype), "moe_gemm_mma: operands not aligned");
   if (em == 0 || num_valid_slots == 0) return B2L_OK;
@@ -224,6 +237,7 @@ extern "C" int b2l_moe_gemm_mma(void* c, const void* a_in, const void* w, const 
   a.slot_weight = (const float*)slot_weight_f32; a.sorted_ids = (const int*)sorted_token_ids;
   a.expert_ids = (const int*)expert_ids; a.num_post = (const int*)num_tokens_post_padded;
   a.num_valid = num_valid_slots; a.top_k = top_k; a.act = act;
+  a.unit = GatedUnit{kUnitClamped, limit, alpha};
   const dim3 grid((unsigned)cdiv64(n, kBN), (unsigned)cdiv64(em, block_size));
   cudaStream_t st = (cudaStream_t)stream;
   if (dtype == B2L_F16) launch_rows<__half, 1>(a, block_size, grid, st);

@@ -5,6 +5,7 @@
 // Every output element is one k-ascending fp32 sum whatever M is, so a token's result does not depend on
 // what else is in the batch.
 #include "common.cuh"
+#include "gated_unit.cuh"
 
 namespace {
 
@@ -56,14 +57,15 @@ __global__ void __launch_bounds__(kThreads) gemm_simt_kernel(T* __restrict__ y, 
   }
 }
 
-// ---- per-head batched product: y[t, h, :] = W[h] . x[t, h, :]  (optionally * sigmoid(gate[t, h])) ------------------
+// ---- per-head batched product: y[t, h, :] = W[h] . x[t, h, :]  (optionally * sigmoid(gate[t, h]), or, with
+// gate_elements, * sigmoid(gate[t, h * n + c]) per element) ----------------------------------------------------------
 // Same tile and the same k-ascending sums as above, blockIdx.z = head.  x / y rows hold the heads side by side
 // (head strides in elements), W is [heads, N, K] dense.
 template <typename T>
 __global__ void __launch_bounds__(kThreads) head_linear_kernel(T* __restrict__ y, const T* __restrict__ x,
                                                                const T* __restrict__ w, const T* __restrict__ gate,
                                                                int64_t m, int64_t n, int64_t k, int64_t xs, int64_t xh,
-                                                               int64_t ys, int64_t yh, int64_t gs) {
+                                                               int64_t ys, int64_t yh, int64_t gs, int gate_elements) {
   pdl_prologue();
   __shared__ float xt[kBK][kBM + 4];
   __shared__ float wt[kBK][kBN + 4];
@@ -100,11 +102,13 @@ __global__ void __launch_bounds__(kThreads) head_linear_kernel(T* __restrict__ y
   for (int i = 0; i < 4; ++i) {
     const int64_t r = m0 + tr + i;
     if (r >= m) continue;
-    const float g = gate ? 1.0f / (1.0f + expf(-to_f32(gate[r * gs + h]))) : 1.0f;
+    float g = (gate && !gate_elements) ? 1.0f / (1.0f + expf(-to_f32(gate[r * gs + h]))) : 1.0f;
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int64_t c = n0 + tc + j;
-      if (c < n) y[r * ys + c] = from_f32<T>(acc[i][j] * g);
+      if (c >= n) continue;
+      if (gate_elements) g = 1.0f / (1.0f + expf(-to_f32(gate[r * gs + h * n + c])));
+      y[r * ys + c] = from_f32<T>(acc[i][j] * g);
     }
   }
 }
@@ -125,7 +129,7 @@ __global__ void __launch_bounds__(kThreads) moe_gemm_simt_kernel(T* __restrict__
                                                                  const int* __restrict__ expert_ids,
                                                                  const int* __restrict__ num_post, int64_t num_valid,
                                                                  int top_k, int64_t n, int64_t k, int64_t as, int64_t cs,
-                                                                 int act) {
+                                                                 int act, GatedUnit unit) {
   pdl_prologue();
   __shared__ float xt[kBK][kGM + 4];
   __shared__ float wt[kBK][kBN + 4];
@@ -175,6 +179,14 @@ __global__ void __launch_bounds__(kThreads) moe_gemm_simt_kernel(T* __restrict__
     const int64_t slot = slot_of[tr + i];
     if (slot >= num_valid) continue;
     const float g = slot_weight ? slot_weight[slot] : 1.0f;
+    if (act == 2) {                                        // columns 2i, 2i + 1 are gate i and up i of a gated unit
+#pragma unroll
+      for (int j = 0; j < 4; j += 2) {
+        const int64_t col = n0 + tc + j;
+        if (col + 1 < n) c[slot * cs + col / 2] = from_f32<T>(unit(acc[i][j], acc[i][j + 1]) * g);
+      }
+      continue;
+    }
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
       const int64_t col = n0 + tc + j;
@@ -205,11 +217,12 @@ extern "C" int b2l_gemm_simt(void* y, const void* x, const void* w, const void* 
   return B2L_OK;
 }
 
-/* y[t, h, :] = W[h] . x[t, h, :] for W [heads, n, k]; gate (nullable) [m, >= heads]: y *= sigmoid(gate[t, h]). */
+/* y[t, h, :] = W[h] . x[t, h, :] for W [heads, n, k]; gate (nullable) [m, >= heads]: y *= sigmoid(gate[t, h]), with
+ * gate_elements [m, >= heads * n]: y[t, h, c] *= sigmoid(gate[t, h * n + c]). */
 extern "C" int b2l_head_linear(void* y, int64_t y_row_stride, int64_t y_head_stride, const void* x,
                                int64_t x_row_stride, int64_t x_head_stride, const void* w, const void* gate,
-                               int64_t gate_row_stride, int64_t m, int heads, int64_t n, int64_t k, int dtype,
-                               void* stream) {
+                               int64_t gate_row_stride, int gate_elements, int64_t m, int heads, int64_t n, int64_t k,
+                               int dtype, void* stream) {
   B2L_REQUIRE(y && x && w, "head_linear: null pointer");
   B2L_REQUIRE(m >= 0 && heads > 0 && heads <= 65535 && n > 0 && k > 0, "head_linear: bad shape");
   if (m == 0) return B2L_OK;
@@ -217,7 +230,8 @@ extern "C" int b2l_head_linear(void* y, int64_t y_row_stride, int64_t y_head_str
   dim3 grid((unsigned)cdiv64(n, kBN), (unsigned)cdiv64(m, kBM), (unsigned)heads);
   B2L_DISPATCH_FLOAT(dtype, "head_linear", {
     b2l_launch(head_linear_kernel<T>, grid, dim3(kThreads), (size_t)0, st, (T*)y, (const T*)x, (const T*)w,
-               (const T*)gate, m, n, k, x_row_stride, x_head_stride, y_row_stride, y_head_stride, gate_row_stride);
+               (const T*)gate, m, n, k, x_row_stride, x_head_stride, y_row_stride, y_head_stride, gate_row_stride,
+               gate ? gate_elements : 0);
   });
   B2L_LAUNCH_CHECK();
   return B2L_OK;
@@ -226,14 +240,16 @@ extern "C" int b2l_head_linear(void* y, int64_t y_row_stride, int64_t y_head_str
 extern "C" int b2l_moe_gemm_simt_block(void) { return kGM; }
 
 /* Grouped product over expert-sorted slots (moe_align_block_size with block_size = b2l_moe_gemm_simt_block()):
- * c[s, :] = act(W[expert(s)] . a[s / top_k, :]) * slot_weight_f32[s];  act: 0 none, 1 exact gelu;  W [experts, n, k]. */
+ * c[s, :] = act(W[expert(s)] . a[s / top_k, :]) * slot_weight_f32[s];  act: 0 none, 1 exact gelu, 2 clamped gated unit
+ * of interleaved rows (2i gate, 2i + 1 up; n / 2 output columns);  W [experts, n, k]. */
 extern "C" int b2l_moe_gemm_simt(void* c, const void* a, const void* w, const void* slot_weight_f32,
                                  const void* sorted_token_ids, const void* expert_ids,
                                  const void* num_tokens_post_padded, int64_t em, int64_t num_valid_slots, int top_k,
-                                 int64_t n, int64_t k, int64_t a_row_stride, int64_t c_row_stride, int act, int dtype,
-                                 void* stream) {
+                                 int64_t n, int64_t k, int64_t a_row_stride, int64_t c_row_stride, int act, float limit,
+                                 float alpha, int dtype, void* stream) {
   B2L_REQUIRE(c && a && w && sorted_token_ids && expert_ids && num_tokens_post_padded, "moe_gemm_simt: null pointer");
-  B2L_REQUIRE(top_k >= 1 && n > 0 && k > 0 && em >= 0 && (act == 0 || act == 1), "moe_gemm_simt: bad shape");
+  B2L_REQUIRE(top_k >= 1 && n > 0 && k > 0 && em >= 0 && act >= 0 && act <= 2 && (act != 2 || n % 2 == 0),
+              "moe_gemm_simt: bad shape");
   if (em == 0 || num_valid_slots == 0) return B2L_OK;
   B2L_REQUIRE(cdiv64(em, kGM) <= 65535, "moe_gemm_simt: %lld row blocks", (long long)cdiv64(em, kGM));
   cudaStream_t st = (cudaStream_t)stream;
@@ -241,7 +257,8 @@ extern "C" int b2l_moe_gemm_simt(void* c, const void* a, const void* w, const vo
   B2L_DISPATCH_FLOAT(dtype, "moe_gemm_simt", {
     b2l_launch(moe_gemm_simt_kernel<T>, grid, dim3(kThreads), (size_t)0, st, (T*)c, (const T*)a, (const T*)w,
                (const float*)slot_weight_f32, (const int*)sorted_token_ids, (const int*)expert_ids,
-               (const int*)num_tokens_post_padded, num_valid_slots, top_k, n, k, a_row_stride, c_row_stride, act);
+               (const int*)num_tokens_post_padded, num_valid_slots, top_k, n, k, a_row_stride, c_row_stride, act,
+               GatedUnit{kUnitClamped, limit, alpha});
   });
   B2L_LAUNCH_CHECK();
   return B2L_OK;

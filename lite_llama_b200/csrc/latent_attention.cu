@@ -7,8 +7,9 @@
 //   a  <- a / rms(a) * wq                in place: the input of the query up-projection
 //   pool row  = [ b / rms(b) * wkv | rotate(r, pos) ]
 //
-//   rope_heads: dst[t, h, :width] = src[t, h, :width] with the first `rot_dims` entries rotated by the token's position
-//               (entry i pairs with entry i + rot_dims/2); the rest is copied.
+//   rope_heads: dst[t, h, :width] = src[t, h, :width] with the first `rot_dims` entries rotated by the token's position;
+//               the rest is copied.
+//   Pairing 1: entry i pairs with entry i + rot_dims/2; 0: neighbours 2i and 2i + 1.
 //
 //   rope_table: cs[t] = [cos(pos_t f_i), i < rot_dims/2 | sin(pos_t f_i)], f_i = base^(-2i/rot_dims), once per step: every
 //               layer with the same rotary constants reads the same table.
@@ -48,7 +49,7 @@ __global__ void __launch_bounds__(128) latent_prepare_kernel(T* __restrict__ pro
                                                              const float* __restrict__ cs_table,
                                                              const T* __restrict__ wq, const T* __restrict__ wkv,
                                                              int64_t tokens, int q_rank, int kv_rank, int rot_dim,
-                                                             int rot_dims, float eps) {
+                                                             int rot_dims, int pairing, float eps) {
   pdl_prologue();
   const int lane = threadIdx.x & 31;
   const int64_t t = (int64_t)blockIdx.x * 4 + (threadIdx.x >> 5);
@@ -69,9 +70,10 @@ __global__ void __launch_bounds__(128) latent_prepare_kernel(T* __restrict__ pro
   const float* cs = cs_table + t * rot_dims;
   for (int i = lane; i < half; i += 32) {
     const float c = cs[i], s = cs[half + i];
-    const float u = to_f32(r[i]), v = to_f32(r[i + half]);
-    dst[kv_rank + i] = from_f32<T>(u * c - v * s);
-    dst[kv_rank + i + half] = from_f32<T>(v * c + u * s);
+    const int e0 = pairing ? i : 2 * i, e1 = pairing ? i + half : 2 * i + 1;
+    const float u = to_f32(r[e0]), v = to_f32(r[e1]);
+    dst[kv_rank + e0] = from_f32<T>(u * c - v * s);
+    dst[kv_rank + e1] = from_f32<T>(v * c + u * s);
   }
   for (int i = 2 * half + lane; i < rot_dim; i += 32) dst[kv_rank + i] = r[i];
 }
@@ -82,7 +84,8 @@ template <typename T>
 __global__ void __launch_bounds__(256) rope_heads_kernel(T* __restrict__ dst, int64_t dst_stride, int dst_head_stride,
                                                          const T* __restrict__ src, int64_t src_stride,
                                                          int src_head_stride, const float* __restrict__ cs_table,
-                                                         int64_t tokens, int heads, int width, int rot_dims) {
+                                                         int64_t tokens, int heads, int width, int rot_dims,
+                                                         int pairing) {
   pdl_prologue();
   const int half = rot_dims / 2, per = width - half;            // items per (token, head): pairs, then the copied tail
   const int64_t idx = (int64_t)blockIdx.x * blockDim.x + threadIdx.x;
@@ -95,9 +98,10 @@ __global__ void __launch_bounds__(256) rope_heads_kernel(T* __restrict__ dst, in
   T* dh = dst + t * dst_stride + (int64_t)h * dst_head_stride;
   if (j < half) {
     const float c = cs_table[t * rot_dims + j], s = cs_table[t * rot_dims + half + j];
-    const float u = to_f32(sh[j]), v = to_f32(sh[j + half]);
-    dh[j] = from_f32<T>(u * c - v * s);
-    dh[j + half] = from_f32<T>(v * c + u * s);
+    const int e0 = pairing ? j : 2 * j, e1 = pairing ? j + half : 2 * j + 1;
+    const float u = to_f32(sh[e0]), v = to_f32(sh[e1]);
+    dh[e0] = from_f32<T>(u * c - v * s);
+    dh[e1] = from_f32<T>(v * c + u * s);
   } else {
     dh[j + half] = sh[j + half];
   }
@@ -120,7 +124,7 @@ extern "C" int b2l_rope_table(void* cos_sin_f32, const void* pos_i32, int64_t to
 extern "C" int b2l_latent_prepare(void* proj, int64_t proj_row_stride, void* pool, int64_t pool_row_stride,
                                   const void* kv_rows_i32, const void* cos_sin_f32, const void* q_norm_weight,
                                   const void* kv_norm_weight, int64_t tokens, int q_rank, int kv_rank, int rot_dim,
-                                  int rot_dims, float eps, int dtype, void* stream) {
+                                  int rot_dims, int pairing, float eps, int dtype, void* stream) {
   B2L_REQUIRE(proj && pool && kv_rows_i32 && q_norm_weight && kv_norm_weight, "latent_prepare: null pointer");
   B2L_REQUIRE(q_rank > 0 && kv_rank > 0 && rot_dim >= 0 && rot_dims >= 0 && rot_dims <= rot_dim && rot_dims % 2 == 0,
               "latent_prepare: bad shape (q_rank %d, kv_rank %d, rot_dim %d, rot_dims %d)", q_rank, kv_rank, rot_dim, rot_dims);
@@ -130,7 +134,7 @@ extern "C" int b2l_latent_prepare(void* proj, int64_t proj_row_stride, void* poo
   B2L_DISPATCH_FLOAT(dtype, "latent_prepare", {
     b2l_launch(latent_prepare_kernel<T>, dim3((unsigned)cdiv64(tokens, 4)), dim3(128), (size_t)0, st, (T*)proj,
                proj_row_stride, (T*)pool, pool_row_stride, (const int*)kv_rows_i32, (const float*)cos_sin_f32,
-               (const T*)q_norm_weight, (const T*)kv_norm_weight, tokens, q_rank, kv_rank, rot_dim, rot_dims, eps);
+               (const T*)q_norm_weight, (const T*)kv_norm_weight, tokens, q_rank, kv_rank, rot_dim, rot_dims, pairing, eps);
   });
   B2L_LAUNCH_CHECK();
   return B2L_OK;
@@ -138,7 +142,7 @@ extern "C" int b2l_latent_prepare(void* proj, int64_t proj_row_stride, void* poo
 
 extern "C" int b2l_rope_heads(void* dst, int64_t dst_row_stride, int dst_head_stride, const void* src,
                               int64_t src_row_stride, int src_head_stride, const void* cos_sin_f32, int64_t tokens,
-                              int heads, int width, int rot_dims, int dtype, void* stream) {
+                              int heads, int width, int rot_dims, int pairing, int dtype, void* stream) {
   B2L_REQUIRE(dst && src, "rope_heads: null pointer");
   B2L_REQUIRE(heads > 0 && width >= 0 && rot_dims >= 0 && rot_dims <= width && rot_dims % 2 == 0,
               "rope_heads: bad shape (heads %d, width %d, rot_dims %d)", heads, width, rot_dims);
@@ -149,7 +153,7 @@ extern "C" int b2l_rope_heads(void* dst, int64_t dst_row_stride, int dst_head_st
     b2l_launch(rope_heads_kernel<T>, dim3((unsigned)cdiv64(tokens * heads * (width - rot_dims / 2), 256)), dim3(256),
                (size_t)0, st, (T*)dst, dst_row_stride,
                dst_head_stride, (const T*)src, src_row_stride, src_head_stride, (const float*)cos_sin_f32, tokens, heads,
-               width, rot_dims);
+               width, rot_dims, pairing);
   });
   B2L_LAUNCH_CHECK();
   return B2L_OK;

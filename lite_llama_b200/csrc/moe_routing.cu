@@ -140,18 +140,19 @@ __global__ void moe_route_kernel(const T* __restrict__ logits, int64_t row_strid
   }
 }
 
-// Sigmoid router with a selection bias and group-limited choice (one CTA per token; the router product is done here,
+// Router with a selection bias and group-limited choice (one CTA per token; the router product is done here,
 // or comes as fp32 logits from a GEMM, in which case the CTA is a single warp):
-//   z = W_r . x (fp32 sums),  s = sigmoid(z),  choice = s + bias
+//   z = W_r . x (fp32 sums),  s = sigmoid(z), or softmax(z) over all experts (`softmax`),  choice = s + bias
 //   the experts form `groups` equal runs of neighbours; a group's score = the sum of its two largest choice scores;
 //   only experts of the `keep` best groups can be chosen; the `top_k` largest choice scores among them win
-//   (lowest index on ties); weights = s of the winners / (their sum + 1e-20), fp32.
+//   (lowest index on ties); weights = scale * s of the winners / (their sum + 1e-20), fp32.
 template <typename T>
 __global__ void __launch_bounds__(128) moe_route_sigmoid_kernel(const T* __restrict__ x, int64_t xs,
                                                                 const T* __restrict__ wr, const T* __restrict__ bias,
                                                                 const float* __restrict__ logits, int num_experts,
                                                                 int k, int top_k, int groups, int keep,
-                                                                int renormalize, float* __restrict__ out_w,
+                                                                int renormalize, int softmax, float scale,
+                                                                float* __restrict__ out_w,
                                                                 int* __restrict__ out_ids) {
   pdl_prologue();
   extern __shared__ float rs[];
@@ -162,7 +163,8 @@ __global__ void __launch_bounds__(128) moe_route_sigmoid_kernel(const T* __restr
   const T* xr = x + (int64_t)t * xs;
   if (logits) {                                  // the router product was done by a GEMM: fp32 logits [tokens, E]
     for (int e = threadIdx.x; e < num_experts; e += blockDim.x) {
-      const float s = 1.0f / (1.0f + expf(-logits[(int64_t)t * num_experts + e]));
+      const float z = logits[(int64_t)t * num_experts + e];
+      const float s = softmax ? z : 1.0f / (1.0f + expf(-z));
       sc[e] = s;
       ch[e] = s + (bias ? to_f32(bias[e]) : 0.f);
     }
@@ -173,12 +175,26 @@ __global__ void __launch_bounds__(128) moe_route_sigmoid_kernel(const T* __restr
     for (int i = lane; i < k; i += 32) acc = fmaf(to_f32(xr[i]), to_f32(w[i]), acc);
     acc = warp_reduce_sum(acc);
     if (lane == 0) {
-      const float s = 1.0f / (1.0f + expf(-acc));
+      const float s = softmax ? acc : 1.0f / (1.0f + expf(-acc));
       sc[e] = s;
       ch[e] = s + (bias ? to_f32(bias[e]) : 0.f);
     }
   }
   __syncthreads();
+  if (softmax) {                                 // every warp reduces the logits itself; then the scores replace them
+    float mx = -INFINITY, sum = 0.f;
+    for (int e = lane; e < num_experts; e += 32) mx = fmaxf(mx, sc[e]);
+    mx = warp_reduce_max(mx);
+    for (int e = lane; e < num_experts; e += 32) sum += expf(sc[e] - mx);
+    sum = warp_reduce_sum(sum);
+    __syncthreads();
+    for (int e = threadIdx.x; e < num_experts; e += blockDim.x) {
+      const float s = expf(sc[e] - mx) / sum;
+      sc[e] = s;
+      ch[e] = s + (bias ? to_f32(bias[e]) : 0.f);
+    }
+    __syncthreads();
+  }
   const int per = num_experts / groups;
   for (int g = threadIdx.x; g < groups; g += blockDim.x) {
     float a = -INFINITY, b = -INFINITY;          // largest, second largest
@@ -240,8 +256,8 @@ __global__ void __launch_bounds__(128) moe_route_sigmoid_kernel(const T* __restr
     }
   }
   __syncwarp();
-  if (!renormalize) return;                      // the weights stay the winners' own scores
-  const float inv = 1.0f / (total + 1e-20f);
+  if (!renormalize && scale == 1.0f) return;     // the weights stay the winners' own scores
+  const float inv = renormalize ? scale / (total + 1e-20f) : scale;
   for (int r = lane; r < top_k; r += 32) out_w[(int64_t)t * top_k + r] *= inv;
 }
 
@@ -300,11 +316,12 @@ extern "C" int b2l_moe_route_topk(void* topk_weights, void* topk_ids_i64, const 
 /* Sigmoid scores + selection bias + group-limited top-k (fp32 throughout).  The router product is done here from
  * x [tokens, k] and router_w [experts, k] in dtype, unless logits_f32 [tokens, experts] brings it; bias [experts] in
  * dtype (nullable); weights_f32 [tokens, top_k], ids_i32 [tokens, top_k].  groups must divide experts; keep <= groups.
- * renormalize 0: the weights are the winners' scores themselves, not divided by their sum. */
+ * renormalize 0: the weights are the winners' scores themselves, not divided by their sum.  softmax: the scores are the
+ * softmax over all experts instead of sigmoids.  scale multiplies the weights. */
 extern "C" int b2l_moe_route_sigmoid_groups(void* weights_f32, void* ids_i32, const void* x, int64_t x_row_stride,
                                             const void* router_w, const void* bias, const void* logits_f32,
                                             int64_t tokens, int num_experts, int64_t k, int top_k, int groups, int keep,
-                                            int renormalize, int dtype, void* stream) {
+                                            int renormalize, int softmax, float scale, int dtype, void* stream) {
   B2L_REQUIRE(weights_f32 && ids_i32 && ((x && router_w) || logits_f32), "moe_route_sigmoid_groups: null pointer");
   B2L_REQUIRE(num_experts > 0 && k > 0 && k < (1ll << 31) && top_k >= 1 && top_k <= num_experts && groups >= 1 &&
                   num_experts % groups == 0 && keep >= 1 && keep <= groups &&
@@ -317,7 +334,7 @@ extern "C" int b2l_moe_route_sigmoid_groups(void* weights_f32, void* ids_i32, co
   B2L_DISPATCH_FLOAT(dtype, "moe_route_sigmoid_groups", {
     b2l_launch(moe_route_sigmoid_kernel<T>, dim3((unsigned)tokens), dim3(logits_f32 ? 32 : 128), smem, st, (const T*)x,
                x_row_stride, (const T*)router_w, (const T*)bias, (const float*)logits_f32, num_experts, (int)k, top_k,
-               groups, keep, renormalize, (float*)weights_f32, (int*)ids_i32);
+               groups, keep, renormalize, softmax, scale, (float*)weights_f32, (int*)ids_i32);
   });
   B2L_LAUNCH_CHECK();
   return B2L_OK;

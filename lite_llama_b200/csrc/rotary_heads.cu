@@ -7,7 +7,8 @@
 //                              RMS-normed over its own head_dim entries with ONE weight [head_dim] shared by the heads
 //                              (nullable = no norm), then its first rot_dims entries are rotated (pairing 0: entries
 //                              2i and 2i+1; pairing 1: entries i and i + rot_dims / 2); q is updated in place, k and v
-//                              go to pool row kv_rows[t] = [k heads | v heads].
+//                              go to pool row kv_rows[t] = [k heads | v heads], v divided by its root mean square per
+//                              head when `v_norm` is set.  kv_heads 0: q alone (a layer that reads another one's cache).
 // Statistics and the rotation are fp32; one rounding to T at the end.
 #include "common.cuh"
 #include "rowvec.cuh"
@@ -30,20 +31,29 @@ __global__ void rope_table_freqs_kernel(float* __restrict__ out, const int* __re
 
 constexpr int kPrepWarps = 4;
 
+// one warp: out = in / sqrt(mean(in^2) + eps)
+template <typename T>
+__device__ __forceinline__ void unit_rms_row(const T* in, T* out, int n, float eps, int lane) {
+  float ss = 0.f;
+  for (int d = lane; d < n; d += 32) { const float v = to_f32(in[d]); ss = fmaf(v, v, ss); }
+  const float r = 1.0f / sqrtf(warp_reduce_sum(ss) / (float)n + eps);
+  for (int d = lane; d < n; d += 32) out[d] = from_f32<T>(to_f32(in[d]) * r);
+}
+
 // One CTA per token, one warp per head at a time.  A head is staged (normed, fp32) in the warp's shared-memory row so
 // that either pairing finds its partner there.
 template <typename T>
 __global__ void __launch_bounds__(kPrepWarps * 32) head_norm_rope_prepare_kernel(
     T* __restrict__ qkv, int64_t qkv_stride, T* __restrict__ pool, int64_t pool_stride, const int* __restrict__ kv_rows,
     const float* __restrict__ cos_sin, const T* __restrict__ q_w, const T* __restrict__ k_w, int H, int G, int D,
-    int Dv, int rot_dims, int pairing, float eps) {
+    int Dv, int rot_dims, int pairing, int v_norm, float eps) {
   pdl_prologue();
   extern __shared__ float stage[];                 // [kPrepWarps][D]
   const int64_t t = blockIdx.x;
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   float* row = stage + warp * D;
   T* src = qkv + t * qkv_stride;
-  T* dst_pool = pool + (int64_t)kv_rows[t] * pool_stride;
+  T* dst_pool = G > 0 ? pool + (int64_t)kv_rows[t] * pool_stride : nullptr;
   const int half = rot_dims / 2;
   const float* cs = cos_sin ? cos_sin + t * rot_dims : nullptr;
   for (int h = warp; h < H + G; h += kPrepWarps) {
@@ -73,26 +83,33 @@ __global__ void __launch_bounds__(kPrepWarps * 32) head_norm_rope_prepare_kernel
     }
     __syncwarp();                                  // the row is reused by the warp's next head
   }
+  if (G == 0) return;
   const T* vin = src + (int64_t)(H + G) * D;
   T* vout = dst_pool + (int64_t)G * D;
+  if (v_norm) {
+    for (int g = (warp + kPrepWarps - (H + G) % kPrepWarps) % kPrepWarps; g < G; g += kPrepWarps)     // continue the warps' round robin
+      unit_rms_row(vin + (int64_t)g * Dv, vout + (int64_t)g * Dv, Dv, eps, lane);
+    return;
+  }
   for (int i = threadIdx.x; i < G * Dv; i += blockDim.x) vout[i] = vin[i];
 }
 
-// The same for the neighbour pairing with 4 elements per access: head_dim a multiple of 4 and at most C * 128, every
-// row and head start aligned to 4 elements.  A lane's 4 elements hold two whole pairs, so the head never leaves the
-// registers: one read and one write per element.
+// The same with 4 elements per access: head_dim a multiple of 4 and at most C * 128, every row and head start aligned to
+// 4 elements.  Neighbour pairing: a lane's 4 elements hold two whole pairs.  Halves pairing (C = 1, rot_dims a multiple
+// of 8): the partners of a lane's 4 elements are the 4 of the lane rot_dims / 8 away.  Either way the head never leaves
+// the registers: one read and one write per element.
 constexpr int kVecWarps = 8;
 
 template <typename T, int C>
 __global__ void __launch_bounds__(kVecWarps * 32) head_norm_rope_prepare_vec_kernel(
     T* __restrict__ qkv, int64_t qkv_stride, T* __restrict__ pool, int64_t pool_stride, const int* __restrict__ kv_rows,
     const float* __restrict__ cos_sin, const T* __restrict__ q_w, const T* __restrict__ k_w, int H, int G, int D,
-    int Dv, int rot_dims, float eps) {
+    int Dv, int rot_dims, int pairing, int v_norm, float eps) {
   pdl_prologue();
   const int64_t t = blockIdx.x;
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   T* src = qkv + t * qkv_stride;
-  T* dst_pool = pool + (int64_t)kv_rows[t] * pool_stride;
+  T* dst_pool = G > 0 ? pool + (int64_t)kv_rows[t] * pool_stride : nullptr;
   const int half = rot_dims / 2;
   const float* cs = cos_sin ? cos_sin + t * rot_dims : nullptr;
   for (int h = warp; h < H + G; h += kVecWarps) {
@@ -115,13 +132,29 @@ __global__ void __launch_bounds__(kVecWarps * 32) head_norm_rope_prepare_vec_ker
 #pragma unroll
     for (int c = 0; c < C; ++c) {
       const int d = (c * 32 + lane) * 4;
-      if (d >= D) continue;
-      if (w) {
+      if (w && d < D) {
         float g[4];
         row_load4(w + d, g);
 #pragma unroll
         for (int e = 0; e < 4; ++e) v[c][e] = v[c][e] * rstd * g[e];
       }
+      if (pairing == 1) {                          // C == 1: every lane of the warp takes part in the exchange
+        const int step = half / 4, first = d < half;
+        float o[4];
+#pragma unroll
+        for (int e = 0; e < 4; ++e) o[e] = __shfl_sync(0xffffffffu, v[c][e], (lane + (first ? step : 32 - step)) & 31);
+        if (cs && d < rot_dims) {
+          const int i0 = first ? d : d - half;
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            const float co = cs[i0 + e], si = cs[half + i0 + e];
+            v[c][e] = first ? v[c][e] * co - o[e] * si : v[c][e] * co + o[e] * si;
+          }
+        }
+        if (d < D) row_store4(out + d, v[c]);
+        continue;
+      }
+      if (d >= D) continue;
 #pragma unroll
       for (int pr = 0; pr < 2; ++pr) {
         const int dd = d + 2 * pr;
@@ -135,8 +168,14 @@ __global__ void __launch_bounds__(kVecWarps * 32) head_norm_rope_prepare_vec_ker
       row_store4(out + d, v[c]);
     }
   }
+  if (G == 0) return;
   const T* vin = src + (int64_t)(H + G) * D;
   T* vout = dst_pool + (int64_t)G * D;
+  if (v_norm) {
+    for (int g = (warp + kVecWarps - (H + G) % kVecWarps) % kVecWarps; g < G; g += kVecWarps)
+      unit_rms_row(vin + (int64_t)g * Dv, vout + (int64_t)g * Dv, Dv, eps, lane);
+    return;
+  }
   if ((G * Dv) % 4 == 0) {
     for (int i = threadIdx.x * 4; i < G * Dv; i += blockDim.x * 4) {
       float x[4];
@@ -167,10 +206,10 @@ extern "C" int b2l_rope_table_freqs(void* cos_sin_f32, const void* pos_i32, cons
 extern "C" int b2l_head_norm_rope_prepare(void* qkv, int64_t qkv_row_stride, void* kv_pool, int64_t kv_row_stride,
                                           const void* kv_rows_i32, const void* cos_sin_f32, const void* q_norm_weight,
                                           const void* k_norm_weight, int64_t tokens, int heads, int kv_heads,
-                                          int head_dim, int v_head_dim, int rot_dims, int pairing, float eps, int dtype,
-                                          void* stream) {
-  B2L_REQUIRE(qkv && kv_pool && kv_rows_i32, "head_norm_rope_prepare: null pointer");
-  B2L_REQUIRE(heads > 0 && kv_heads > 0 && head_dim > 0 && v_head_dim > 0, "head_norm_rope_prepare: bad shape");
+                                          int head_dim, int v_head_dim, int rot_dims, int pairing, int v_norm, float eps,
+                                          int dtype, void* stream) {
+  B2L_REQUIRE(qkv && (kv_heads == 0 || (kv_pool && kv_rows_i32)), "head_norm_rope_prepare: null pointer");
+  B2L_REQUIRE(heads > 0 && kv_heads >= 0 && head_dim > 0 && v_head_dim > 0, "head_norm_rope_prepare: bad shape");
   B2L_REQUIRE(rot_dims >= 0 && rot_dims % 2 == 0 && rot_dims <= head_dim && (rot_dims == 0 || cos_sin_f32),
               "head_norm_rope_prepare: %d rotated entries of %d", rot_dims, head_dim);
   B2L_REQUIRE(pairing == 0 || pairing == 1, "head_norm_rope_prepare: pairing %d", pairing);
@@ -182,9 +221,10 @@ extern "C" int b2l_head_norm_rope_prepare(void* qkv, int64_t qkv_row_stride, voi
   b2l_launch(head_norm_rope_prepare_vec_kernel<T, CV>, dim3((unsigned)tokens), dim3(kVecWarps * 32), (size_t)0, st, \
              (T*)qkv, qkv_row_stride, (T*)kv_pool, kv_row_stride, (const int*)kv_rows_i32,                          \
              (const float*)cos_sin_f32, (const T*)q_norm_weight, (const T*)k_norm_weight, heads, kv_heads, head_dim, \
-             v_head_dim, rot_dims, eps)
+             v_head_dim, rot_dims, pairing, v_norm, eps)
   B2L_DISPATCH_FLOAT(dtype, "head_norm_rope_prepare", {
-    const bool vec = pairing == 0 && head_dim % 4 == 0 && head_dim <= 256 && qkv_row_stride % 4 == 0 &&
+    const bool vec = (pairing == 0 || (head_dim <= 128 && rot_dims % 8 == 0)) && head_dim % 4 == 0 && head_dim <= 256 &&
+                     qkv_row_stride % 4 == 0 &&
                      kv_row_stride % 4 == 0 && row_aligned4<T>(qkv) && row_aligned4<T>(kv_pool) &&
                      row_aligned4<T>(q_norm_weight) && row_aligned4<T>(k_norm_weight) &&
                      ((kv_heads * v_head_dim) % 4 != 0 || ((int64_t)(heads + kv_heads) * head_dim) % 4 == 0);
@@ -193,7 +233,7 @@ extern "C" int b2l_head_norm_rope_prepare(void* qkv, int64_t qkv_row_stride, voi
     b2l_launch(head_norm_rope_prepare_kernel<T>, dim3((unsigned)tokens), dim3(kPrepWarps * 32), smem, st, (T*)qkv,
                qkv_row_stride, (T*)kv_pool, kv_row_stride, (const int*)kv_rows_i32, (const float*)cos_sin_f32,
                (const T*)q_norm_weight, (const T*)k_norm_weight, heads, kv_heads, head_dim, v_head_dim, rot_dims,
-               pairing, eps);
+               pairing, v_norm, eps);
   });
 #undef B2L_PREP_VEC
   B2L_LAUNCH_CHECK();

@@ -4,7 +4,9 @@
 //
 //   causal_conv_silu      (`activation` 1; 0 = the plain convolution) out[t, c] = silu(bias[c] + sum_j w[c, K-1-j] * in[t-j, c]); inputs before the step come from
 //                         the slot's conv tail (the last K-1 inputs), inputs before the sequence are zero
-//   conv_tail_update      the slot's conv tail after the step (in place)
+//                         (`residual`: out = in + that).  The slot's conv tail is advanced in place by the same launch:
+//                         the first taps - 1 tokens of a sequence (the only readers of its old tail) belong to one thread
+//                         per channel, which stores the new tail afterwards
 //   ssm_scan              dt = softplus(dt_raw + dt_bias); S <- exp(-exp(A_log) dt) S + dt B x^T; y = S^T C + D x
 //                         S in fp32 registers for the whole step, read from / written to the slot once
 //                         (slot layout [head, n, p]).  With `fixed_decay` (fp32 per head) the same kernel runs a
@@ -31,108 +33,122 @@ __device__ __forceinline__ int find_seq(const int* __restrict__ seq_start, int n
 
 template <typename T>
 __global__ void causal_conv_silu_kernel(T* __restrict__ out, const T* __restrict__ in, int64_t in_stride,
-                                        const T* __restrict__ w, const T* __restrict__ bias,
-                                        const T* __restrict__ tail, const int* __restrict__ seq_start,
-                                        const int* __restrict__ seq_ctx, const int* __restrict__ seq_slot, int nseq,
-                                        int channels, int taps, int act) {
+                                        const T* __restrict__ w, const T* __restrict__ bias, T* tail,
+                                        const int* __restrict__ seq_start, const int* __restrict__ seq_ctx,
+                                        const int* __restrict__ seq_slot, int nseq, int channels, int taps, int act,
+                                        int residual) {
   pdl_prologue();
-  const int tok = blockIdx.y;
-  const int s = find_seq(seq_start, nseq, tok);
-  const int local = tok - seq_start[s], ctx = seq_ctx[s];
+  const int tok0 = blockIdx.y;
+  const int s = find_seq(seq_start, nseq, tok0);
+  const int start = seq_start[s], len = seq_start[s + 1] - start, ctx = seq_ctx[s], local0 = tok0 - start;
   const int64_t slot = seq_slot[s];
   const int c = blockIdx.x * blockDim.x + threadIdx.x;
-  if (c >= channels) return;
-  float acc = to_f32(bias[c]);
-  for (int j = 0; j < taps; ++j) {                 // j tokens back
-    const int i = local - j;
-    float v = 0.f;
-    if (i >= 0) v = to_f32(in[(int64_t)(tok - j) * in_stride + c]);
-    else if (ctx + i >= 0) v = to_f32(tail[(slot * (taps - 1) + (taps - 1 + i)) * channels + c]);
-    acc = fmaf(to_f32(w[(int64_t)c * taps + (taps - 1 - j)]), v, acc);
+  if (c >= channels || (local0 > 0 && local0 < taps - 1)) return;
+  const int reps = local0 == 0 ? max(1, min(len, taps - 1)) : 1;
+  for (int r = 0; r < reps; ++r) {
+    const int tok = tok0 + r, local = local0 + r;
+    float acc = bias ? to_f32(bias[c]) : 0.f;
+    if (residual) acc += to_f32(in[(int64_t)tok * in_stride + c]);
+    for (int j = 0; j < taps; ++j) {               // j tokens back
+      const int i = local - j;
+      float v = 0.f;
+      if (i >= 0) v = to_f32(in[(int64_t)(tok - j) * in_stride + c]);
+      else if (ctx + i >= 0) v = to_f32(tail[(slot * (taps - 1) + (taps - 1 + i)) * channels + c]);
+      acc = fmaf(to_f32(w[(int64_t)c * taps + (taps - 1 - j)]), v, acc);
+    }
+    out[(int64_t)tok * channels + c] = from_f32<T>(act ? silu_f(acc) : acc);
   }
-  out[(int64_t)tok * channels + c] = from_f32<T>(act ? silu_f(acc) : acc);
+  if (local0 > 0 || taps == 1) return;
+  // tail entry j holds the input at index ctx + len - (taps - 1) + j; ascending j only reads later entries of the old one
+  T* mine = tail + slot * (taps - 1) * channels;
+  for (int j = 0; j < taps - 1; ++j) {
+    const int p = ctx + len - (taps - 1) + j;
+    T v = from_f32<T>(0.f);
+    if (p >= ctx) v = in[(int64_t)(start + p - ctx) * in_stride + c];
+    else if (p >= 0) v = mine[(int64_t)(j + len) * channels + c];
+    mine[(int64_t)j * channels + c] = v;
+  }
 }
 
 // The same with 16-byte accesses: one thread = VEC consecutive channels (channels, the input row stride and the
 // column window's start all multiples of VEC elements).
 template <typename T, int TAPS>     // TAPS > 0: tap count known at compile time, weights held in registers
 __global__ void causal_conv_silu_vec_kernel(T* __restrict__ out, const T* __restrict__ in, int64_t in_stride,
-                                            const T* __restrict__ w, const T* __restrict__ bias,
-                                            const T* __restrict__ tail, const int* __restrict__ seq_start,
-                                            const int* __restrict__ seq_ctx, const int* __restrict__ seq_slot,
-                                            int nseq, int channels, int taps, int act) {
+                                            const T* __restrict__ w, const T* __restrict__ bias, T* tail,
+                                            const int* __restrict__ seq_start, const int* __restrict__ seq_ctx,
+                                            const int* __restrict__ seq_slot, int nseq, int channels, int taps, int act,
+                                            int residual) {
   pdl_prologue();
   constexpr int VEC = 16 / (int)sizeof(T);
-  const int tok = blockIdx.y;
-  const int s = find_seq(seq_start, nseq, tok);
-  const int local = tok - seq_start[s], ctx = seq_ctx[s];
+  const int tok0 = blockIdx.y;
+  const int s = find_seq(seq_start, nseq, tok0);
+  const int start = seq_start[s], len = seq_start[s + 1] - start, ctx = seq_ctx[s], local0 = tok0 - start;
   const int64_t slot = seq_slot[s];
   const int c = (blockIdx.x * blockDim.x + threadIdx.x) * VEC;
-  if (c >= channels) return;
-  float acc[VEC];
-  {
-    const uint4 raw = ldg_128(bias + c);
-    const T* e = reinterpret_cast<const T*>(&raw);
+  if (c >= channels || (local0 > 0 && local0 < taps - 1)) return;
+  const int reps = local0 == 0 ? max(1, min(len, taps - 1)) : 1;
+  for (int rep = 0; rep < reps; ++rep) {
+    const int tok = tok0 + rep, local = local0 + rep;
+    float acc[VEC];
 #pragma unroll
-    for (int k = 0; k < VEC; ++k) acc[k] = to_f32(e[k]);
+    for (int k = 0; k < VEC; ++k) acc[k] = 0.f;
+    if (bias) {
+      const uint4 raw = ldg_128(bias + c);
+      const T* e = reinterpret_cast<const T*>(&raw);
+#pragma unroll
+      for (int k = 0; k < VEC; ++k) acc[k] = to_f32(e[k]);
+    }
+    if (residual) {
+      const uint4 raw = ldg_128(in + (int64_t)tok * in_stride + c);
+      const T* e = reinterpret_cast<const T*>(&raw);
+#pragma unroll
+      for (int k = 0; k < VEC; ++k) acc[k] += to_f32(e[k]);
+    }
+    if (TAPS > 0) {
+      // the VEC channels' taps are VEC * TAPS consecutive elements = TAPS 16-byte vectors
+      float wf[VEC * (TAPS > 0 ? TAPS : 1)];
+#pragma unroll
+      for (int v = 0; v < TAPS; ++v) {
+        const uint4 raw = ldg_128(w + (int64_t)c * TAPS + v * VEC);
+        const T* e = reinterpret_cast<const T*>(&raw);
+#pragma unroll
+        for (int k = 0; k < VEC; ++k) wf[v * VEC + k] = to_f32(e[k]);
+      }
+#pragma unroll
+      for (int j = 0; j < TAPS; ++j) {
+        const int i = local - j;
+        uint4 raw = make_uint4(0u, 0u, 0u, 0u);
+        if (i >= 0) raw = ldg_128(in + (int64_t)(tok - j) * in_stride + c);
+        else if (ctx + i >= 0) raw = ldg_128(tail + (slot * (TAPS - 1) + (TAPS - 1 + i)) * channels + c);
+        const T* e = reinterpret_cast<const T*>(&raw);
+#pragma unroll
+        for (int k = 0; k < VEC; ++k) acc[k] = fmaf(wf[k * TAPS + (TAPS - 1 - j)], to_f32(e[k]), acc[k]);
+      }
+    } else {
+      for (int j = 0; j < taps; ++j) {
+        const int i = local - j;
+        uint4 raw = make_uint4(0u, 0u, 0u, 0u);
+        if (i >= 0) raw = ldg_128(in + (int64_t)(tok - j) * in_stride + c);
+        else if (ctx + i >= 0) raw = ldg_128(tail + (slot * (taps - 1) + (taps - 1 + i)) * channels + c);
+        const T* e = reinterpret_cast<const T*>(&raw);
+#pragma unroll
+        for (int k = 0; k < VEC; ++k) acc[k] = fmaf(to_f32(w[(int64_t)(c + k) * taps + (taps - 1 - j)]), to_f32(e[k]), acc[k]);
+      }
+    }
+    uint4 res;
+    T* e = reinterpret_cast<T*>(&res);
+#pragma unroll
+    for (int k = 0; k < VEC; ++k) e[k] = from_f32<T>(act ? silu_f(acc[k]) : acc[k]);
+    *reinterpret_cast<uint4*>(out + (int64_t)tok * channels + c) = res;
   }
-  if (TAPS > 0) {
-    // the VEC channels' taps are VEC * TAPS consecutive elements = TAPS 16-byte vectors
-    float wf[VEC * (TAPS > 0 ? TAPS : 1)];
-#pragma unroll
-    for (int v = 0; v < TAPS; ++v) {
-      const uint4 raw = ldg_128(w + (int64_t)c * TAPS + v * VEC);
-      const T* e = reinterpret_cast<const T*>(&raw);
-#pragma unroll
-      for (int k = 0; k < VEC; ++k) wf[v * VEC + k] = to_f32(e[k]);
-    }
-#pragma unroll
-    for (int j = 0; j < TAPS; ++j) {
-      const int i = local - j;
-      uint4 raw = make_uint4(0u, 0u, 0u, 0u);
-      if (i >= 0) raw = ldg_128(in + (int64_t)(tok - j) * in_stride + c);
-      else if (ctx + i >= 0) raw = ldg_128(tail + (slot * (TAPS - 1) + (TAPS - 1 + i)) * channels + c);
-      const T* e = reinterpret_cast<const T*>(&raw);
-#pragma unroll
-      for (int k = 0; k < VEC; ++k) acc[k] = fmaf(wf[k * TAPS + (TAPS - 1 - j)], to_f32(e[k]), acc[k]);
-    }
-  } else {
-    for (int j = 0; j < taps; ++j) {
-      const int i = local - j;
-      uint4 raw = make_uint4(0u, 0u, 0u, 0u);
-      if (i >= 0) raw = ldg_128(in + (int64_t)(tok - j) * in_stride + c);
-      else if (ctx + i >= 0) raw = ldg_128(tail + (slot * (taps - 1) + (taps - 1 + i)) * channels + c);
-      const T* e = reinterpret_cast<const T*>(&raw);
-#pragma unroll
-      for (int k = 0; k < VEC; ++k) acc[k] = fmaf(to_f32(w[(int64_t)(c + k) * taps + (taps - 1 - j)]), to_f32(e[k]), acc[k]);
-    }
-  }
-  uint4 res;
-  T* e = reinterpret_cast<T*>(&res);
-#pragma unroll
-  for (int k = 0; k < VEC; ++k) e[k] = from_f32<T>(act ? silu_f(acc[k]) : acc[k]);
-  *reinterpret_cast<uint4*>(out + (int64_t)tok * channels + c) = res;
-}
-
-template <typename T>
-__global__ void conv_tail_update_kernel(T* __restrict__ tail, const T* __restrict__ in, int64_t in_stride,
-                                        const int* __restrict__ seq_start, const int* __restrict__ seq_ctx,
-                                        const int* __restrict__ seq_slot, int channels, int taps) {
-  pdl_prologue();
-  const int s = blockIdx.y;
-  const int start = seq_start[s], len = seq_start[s + 1] - start, ctx = seq_ctx[s];
-  const int64_t slot = seq_slot[s];
-  const int c = blockIdx.x * blockDim.x + threadIdx.x;
-  if (c >= channels || len <= 0) return;
-  const int keep = taps - 1;
-  T* mine = tail + slot * keep * channels;
-  // entry j holds the input at absolute index ctx + len - keep + j; ascending j only reads entries > j of the old tail
-  for (int j = 0; j < keep; ++j) {
-    const int a = ctx + len - keep + j;
-    T v = from_f32<T>(0.f);
-    if (a >= ctx) v = in[(int64_t)(start + a - ctx) * in_stride + c];
-    else if (a >= 0) v = mine[(int64_t)(j + len) * channels + c];
-    mine[(int64_t)j * channels + c] = v;
+  if (local0 > 0 || taps == 1) return;
+  T* mine = tail + slot * (taps - 1) * channels;
+  for (int j = 0; j < taps - 1; ++j) {
+    const int p = ctx + len - (taps - 1) + j;
+    uint4 v = make_uint4(0u, 0u, 0u, 0u);
+    if (p >= ctx) v = ldg_128(in + (int64_t)(start + p - ctx) * in_stride + c);
+    else if (p >= 0) v = *reinterpret_cast<const uint4*>(mine + (int64_t)(j + len) * channels + c);
+    *reinterpret_cast<uint4*>(mine + (int64_t)j * channels + c) = v;
   }
 }
 
@@ -458,18 +474,17 @@ __global__ void gated_group_norm_vec_kernel(T* __restrict__ o, const float* __re
 extern "C" int b2l_causal_conv_silu(void* out, const void* in, int64_t in_row_stride, const void* weight,
                                     const void* bias, void* tail, const void* seq_start, const void* seq_ctx,
                                     const void* seq_slot, int64_t num_seqs, int64_t tokens, int channels, int taps,
-                                    int activation, int dtype, void* stream) {
-  B2L_REQUIRE(out && in && weight && bias && (tail || taps == 1) && seq_start && seq_ctx && seq_slot, "causal_conv_silu: null pointer");
+                                    int activation, int residual, int dtype, void* stream) {
+  B2L_REQUIRE(out && in && weight && (tail || taps == 1) && seq_start && seq_ctx && seq_slot, "causal_conv_silu: null pointer");
   B2L_REQUIRE(channels > 0 && taps >= 1 && num_seqs >= 0 && tokens >= 0, "causal_conv_silu: bad shape");
   if (tokens == 0 || num_seqs == 0) return B2L_OK;
   cudaStream_t st = (cudaStream_t)stream;
   const dim3 block(128), grid((unsigned)cdiv64(channels, 128), (unsigned)tokens);
-  const dim3 grid2((unsigned)cdiv64(channels, 128), (unsigned)num_seqs);
 #define B2L_CONV(TP)                                                                                                 \
   b2l_launch(causal_conv_silu_vec_kernel<T, TP>, dim3((unsigned)cdiv64(channels / VEC, 128), (unsigned)tokens), block, \
-             (size_t)0, st, (T*)out, (const T*)in, in_row_stride, (const T*)weight, (const T*)bias, (const T*)tail,  \
+             (size_t)0, st, (T*)out, (const T*)in, in_row_stride, (const T*)weight, (const T*)bias, (T*)tail,        \
              (const int*)seq_start, (const int*)seq_ctx, (const int*)seq_slot, (int)num_seqs, channels, taps,        \
-             activation)
+             activation, residual)
   B2L_DISPATCH_FLOAT(dtype, "causal_conv_silu", {
     constexpr int VEC = 16 / (int)sizeof(T);
     const bool vec = channels % VEC == 0 && in_row_stride % VEC == 0 && (uintptr_t)in % 16 == 0 &&
@@ -481,12 +496,8 @@ extern "C" int b2l_causal_conv_silu(void* out, const void* in, int64_t in_row_st
     else if (vec) B2L_CONV(0);
     else
       b2l_launch(causal_conv_silu_kernel<T>, grid, block, (size_t)0, st, (T*)out, (const T*)in, in_row_stride,
-                 (const T*)weight, (const T*)bias, (const T*)tail, (const int*)seq_start, (const int*)seq_ctx,
-                 (const int*)seq_slot, (int)num_seqs, channels, taps, activation);
-    b2l_count_launch();
-    if (taps > 1)
-      b2l_launch(conv_tail_update_kernel<T>, grid2, block, (size_t)0, st, (T*)tail, (const T*)in, in_row_stride,
-                 (const int*)seq_start, (const int*)seq_ctx, (const int*)seq_slot, channels, taps);
+                 (const T*)weight, (const T*)bias, (T*)tail, (const int*)seq_start, (const int*)seq_ctx,
+                 (const int*)seq_slot, (int)num_seqs, channels, taps, activation, residual);
   });
 #undef B2L_CONV
   B2L_LAUNCH_CHECK();

@@ -86,7 +86,7 @@ class Engine:
         """Pool rows a sequence of ``tokens`` holds at most: all of them, or -- when every cached layer has a sliding
         window and the runner gives unseen rows back on the way -- what the windows keep plus one portion."""
         keep = getattr(self.runner, "keep_positions", 0)
-        return min(tokens, keep + self.max_portion) if keep else tokens
+        return min(tokens, keep + getattr(self.runner, "keep_first", 0) + self.max_portion) if keep else tokens
 
     def has_work(self) -> bool:
         return bool(self.waiting or self.running)

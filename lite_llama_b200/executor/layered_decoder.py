@@ -29,6 +29,13 @@ Designs registered here:
     short convolution, and softmax attention (biased projections, per-head q / k norm, neighbour-paired rotary
     positions with frequency interpolation by parts, soft cap, block-diagonal causal mask) side by side with decayed
     linear attention.
+  * ``Gofezen``: one-norm parallel blocks; forget-gate linear attention, convolved window attention with mixed heads
+    beside a gated delta rule, gated routed experts.
+  * ``Torutar``: a residual of several streams (hyper-connections) that every sublayer reads as a weighted sum and writes
+    all at once, a causal convolution on what a sublayer reads and a logistic gate on what it returns; mixers: a matrix
+    memory with exponential gates, window attention with kept first tokens, sinks and head gates (some layers read
+    another layer's cache), latent attention with an element-wise output gate; clamped gated experts behind a softmax
+    router.
 """
 
 from __future__ import annotations
@@ -57,6 +64,7 @@ from ..kernels import (
     head_norm_rope_prepare,
     latent_prepare,
     linear,
+    mlstm,
     norm_sigmoid_gate,
     post_norm_residual,
     relu_squared,
@@ -71,12 +79,15 @@ from ..kernels import (
     MIXED_HEAD_MAX_KEYS,
     softcap_to_f32,
     ssm_scan,
+    stream_embed,
+    stream_mix,
     swiglu_forward,
     swiglu_scaled,
 )
 from .model_config import (BlockAttentionSpec, ConvWindowAttentionSpec, DecayAttentionSpec, DeltaRuleSpec, DenseMlpSpec,
                            ForgetGateAttentionSpec, LatentAttentionSpec, LayeredConfig, LayerSpec, Mamba2Spec,
-                           MinGruSpec, MoeMlpSpec, RgLruSpec, SideBySideSpec, SinkAttentionSpec, WindowDeltaPairSpec)
+                           MinGruSpec, MlstmSpec, MoeMlpSpec, RgLruSpec, SideBySideSpec, SinkAttentionSpec,
+                           WindowAttentionSpec, WindowDeltaPairSpec)
 from .ragged_batch import RaggedBatch
 from .registry import Architecture, register
 
@@ -94,6 +105,9 @@ class LayeredLayerWeights:
     ls2: torch.Tensor | None = None
     side: dict[str, torch.Tensor] | None = None          # per-layer token input: gate, proj, norm
     depth: torch.Tensor | None = None                    # depth-average coefficients over [embedding, layer results]
+    # stream designs, one dict per sublayer (mixer, feed-forward): read coefficients "in" [streams], write coefficients
+    # "coef" [out | mix] (both fp32), "norm", input convolution "conv", result gate "gate", "gate_b"
+    subs: list[dict[str, torch.Tensor]] | None = None
 
 
 @dataclass
@@ -105,6 +119,7 @@ class LayeredWeights:
     layers: list[LayeredLayerWeights] = field(default_factory=list)
     embed_norm: torch.Tensor | None = None
     side_embed: torch.Tensor | None = None               # [vocab, layers * token_side_dim]
+    stream_ones: torch.Tensor | None = None              # fp32 ones [streams]: the output reads the sum of the streams
 
     def nbytes_per_step(self) -> int:
         """Weight bytes one step streams (embedding / position gathers excluded)."""
@@ -114,7 +129,7 @@ class LayeredWeights:
             if id(lw) in seen:                           # a layer that shares another one's weights
                 continue
             seen.add(id(lw))
-            for d in (lw.mix, lw.mlp or {}, lw.side or {}):
+            for d in (lw.mix, lw.mlp or {}, lw.side or {}, *(lw.subs or [])):
                 total += sum(t.numel() * t.element_size() for t in d.values())
         return total
 
@@ -222,20 +237,22 @@ def latent_attention_mixer(li: int, spec: LatentAttentionSpec, w: dict[str, torc
     norms, rotation and the cache write (``latent_prepare``) -> query up-projection -> the queries' unrotated parts
     multiplied into the latent space per head (``W_uk^T q``), their rotated parts turned by the position -> attention
     over the cached rows [latent | rotated key part] as ONE key/value head whose values are the latent itself (sliding
-    window) -> per-head value up-projection with the sigmoid gate in its epilogue -> output projection.  Equal to
+    window) -> per-head value up-projection with the sigmoid gate (one per head, or per element) in its epilogue ->
+    output projection.  Equal to
     expanding per-head keys and values from the latent for every cached token, without doing so."""
     b = ctx.batch
     H, dim, rot, rank = spec.heads, spec.head_dim, spec.rot_dim, spec.kv_rank
     proj = linear(x, w["down"])
     pool = ctx.kv_buffer[li]
     cos_sin = ctx.rope(spec.rot_dims, spec.rot_base)
-    latent_prepare(proj, pool, b.kv_rows, cos_sin, w["q_norm"], w["kv_norm"], spec.q_rank, rank, rot, spec.rot_dims, eps)
+    latent_prepare(proj, pool, b.kv_rows, cos_sin, w["q_norm"], w["kv_norm"], spec.q_rank, rank, rot, spec.rot_dims, eps,
+                   spec.pairing)
     q = linear(proj[:, :spec.q_rank], w["uq"])
     D = rank + rot
     qa = torch.empty((b.tokens, H * D), dtype=q.dtype, device=q.device)
     head_linear(qa, D, q, dim + rot, w["uk_t"])
     if rot:
-        rope_heads(qa[:, rank:], D, q[:, dim:], dim + rot, cos_sin, H, rot, spec.rot_dims)
+        rope_heads(qa[:, rank:], D, q[:, dim:], dim + rot, cos_sin, H, rot, spec.rot_dims, spec.pairing)
     lat = torch.empty((b.tokens, H * rank), dtype=q.dtype, device=q.device)
     common = (H, 1, D, rank, spec.scale, 0.0)
     if b.num_portions:
@@ -248,7 +265,7 @@ def latent_attention_mixer(li: int, spec: LatentAttentionSpec, w: dict[str, torc
                        None, *common, num_splits=splits, split_keys=per, window=spec.window, v_col0=0)
     out = torch.empty((b.tokens, H * spec.v_head_dim), dtype=q.dtype, device=q.device)
     gate = proj[:, spec.q_rank + rank + rot:] if spec.out_gate else None
-    head_linear(out, spec.v_head_dim, lat, rank, w["uv"], gate)
+    head_linear(out, spec.v_head_dim, lat, rank, w["uv"], gate, spec.element_gate)
     return linear(out, w["o"])
 
 
@@ -420,6 +437,58 @@ def window_delta_mixer(li: int, spec: WindowDeltaPairSpec, w: dict[str, torch.Te
     return Branches(left, None, right, None, spec.left_scale, spec.right_scale)
 
 
+def aligned_columns(*sizes: int) -> list[int]:
+    """Start columns of parts laid side by side in one row, each start a multiple of 8 (16-byte accesses); the last entry
+    is the row's padded width."""
+    starts, at = [], 0
+    for n in sizes:
+        starts.append(at)
+        at += -(-n // 8) * 8
+    return [*starts, at]
+
+
+def window_attention_mixer(li: int, spec: WindowAttentionSpec, w: dict[str, torch.Tensor], x: torch.Tensor,
+                           ctx: StepContext, eps: float) -> torch.Tensor:
+    """ONE biased projection [q | k | v | pad | head gates] (a layer that reads another layer's cache: [q | pad | head
+    gates]) -> per-head norms, rotation, value norm and the cache write in one kernel -> attention over the pool (window
+    with kept first positions, sink, head gate in the epilogue) -> biased out-projection."""
+    b, H, D, Dv = ctx.batch, spec.heads, spec.head_dim, spec.v_head_dim
+    own = spec.kv_from is None
+    G = spec.kv_heads if own else 0
+    proj = linear(x, w["in"], w["in_b"])
+    pool = ctx.kv_buffer[li if own else spec.kv_from]
+    cos_sin = ctx.rope(spec.rot_dims, spec.rot_base)
+    head_norm_rope_prepare(proj, pool if own else None, b.kv_rows, cos_sin, w["q_norm"], w.get("k_norm"), H, G, D, Dv,
+                           spec.rot_dims, eps, spec.pairing, spec.v_norm)
+    g0 = aligned_columns(H * D + G * (D + Dv))[1]
+    gate = proj[:, g0:g0 + H] if spec.head_gate else None
+    att = torch.empty((b.tokens, H * Dv), dtype=proj.dtype, device=proj.device)
+    common = (H, spec.kv_heads, D, Dv, spec.scale, 0.0)
+    mask = dict(window=spec.window, keep_first=spec.keep_first, gate=gate)
+    if b.num_portions:
+        sink_attention(att, proj, pool, ctx.table, b.seq_start, b.seq_ctx, b.seq_slot, b.portion_list, b.num_portions,
+                       b.max_portion, w.get("sink"), *common, **mask)
+    if b.num_singles:
+        keys = b.max_single_ctx + 1
+        splits, per = split_plan(min(keys, spec.window + spec.keep_first) if spec.window else keys)
+        sink_attention(att, proj, pool, ctx.table, b.seq_start, b.seq_ctx, b.seq_slot, b.single_list, b.num_singles, 1,
+                       w.get("sink"), *common, num_splits=splits, split_keys=per, **mask)
+    return linear(att, w["o"], w["o_b"])
+
+
+def mlstm_mixer(li: int, spec: MlstmSpec, w: dict[str, torch.Tensor], x: torch.Tensor, ctx: StepContext,
+                eps: float) -> torch.Tensor:
+    """ONE projection [q | k | v | gate | input-gate logits | forget-gate logits] (parts start on 16 bytes) -> the
+    recurrence against the slot's fp32 memory, normaliser and log scale (gates in fp32 inside the kernel) -> per-head RMS
+    norm and the element-wise logistic gate -> out-projection."""
+    H, D, V = spec.heads, spec.head_dim, spec.v_head_dim
+    proj = linear(x, w["in"])
+    q0, k0, v0, g0, i0, f0, _ = aligned_columns(H * D, H * D, H * V, H * V, H, H)
+    y = mlstm(ctx.states.ssm_state[li], proj[:, q0:q0 + H * D], proj[:, k0:k0 + H * D], proj[:, v0:v0 + H * V],
+              proj[:, i0:i0 + H], proj[:, f0:f0 + H], w["i_b"], w["f_b"], ctx.batch, H, D, V, spec.gate_cap, D ** -0.5)
+    return linear(head_norm_gate(y, w["norm"], H, eps, proj[:, g0:g0 + H * V], "sigmoid"), w["o"])
+
+
 def spec_magnitude(spec: BlockAttentionSpec) -> float:
     return rotary_frequencies(spec.rot_dims, spec.rot_base, spec.rot_factor, spec.rot_original, spec.rot_fast,
                               spec.rot_slow)[1]
@@ -435,7 +504,7 @@ def _activate(kind: str, x: torch.Tensor) -> torch.Tensor:
     raise ValueError(f"unknown feed-forward activation {kind!r}")
 
 
-def dense_feed_forward(spec: DenseMlpSpec, w: dict[str, torch.Tensor], x: torch.Tensor) -> torch.Tensor:
+def dense_feed_forward(spec: DenseMlpSpec, w: dict[str, torch.Tensor], x: torch.Tensor, reduce: bool = True) -> torch.Tensor:
     if spec.gated:                                   # [gate | up] is one product; silu(gate) * up one kernel
         if spec.activation != "silu":
             raise ValueError(f"unknown gated feed-forward activation {spec.activation!r}")
@@ -444,12 +513,36 @@ def dense_feed_forward(spec: DenseMlpSpec, w: dict[str, torch.Tensor], x: torch.
     return linear(_activate(spec.activation, linear(x, w["up"])), w["down"])
 
 
-def moe_feed_forward(spec: MoeMlpSpec, w: dict[str, torch.Tensor], x: torch.Tensor) -> torch.Tensor:
-    """Router (product, sigmoid, bias, group-limited top-k: one launch) -> the shared expert as two dense products ->
-    the routed experts as two grouped products; the shared expert's output joins the weighted sum in its kernel."""
+@dataclass
+class ExpertTerms:
+    """A feed-forward's output as the rows its consumer sums: the chosen experts' weighted outputs ``[tokens, top, n]`` and
+    the shared expert's ``[tokens, n]``."""
+
+    terms: torch.Tensor
+    addend: torch.Tensor | None
+
+
+def moe_feed_forward(spec: MoeMlpSpec, w: dict[str, torch.Tensor], x: torch.Tensor,
+                     reduce: bool = True) -> torch.Tensor | ExpertTerms:
+    """Router (product, scores, bias, group-limited top-k) -> the shared expert as two dense products ->
+    the routed experts as two grouped products; the shared expert's output joins the weighted sum in its kernel
+    (``reduce=False``: the terms are handed out for the consumer to sum)."""
     weights, ids = route_sigmoid_groups(x, w["router"], w.get("correction"), spec.top, spec.groups, spec.keep,
-                                        renormalize=spec.renormalize)
+                                        renormalize=spec.renormalize, scores=spec.scores, scale=spec.scale)
     shared = None
+    if spec.activation == "clamped":
+        # the unit is formed in the grouped product's epilogue (gate and up rows interleaved); the shared expert's
+        # [gate | up] is one dense product with the unit as a kernel of its own
+        if spec.shared_ff:
+            f = spec.shared_ff
+            gu = linear(x, w["shared_gate_up"])
+            shared = linear(swiglu_scaled(gu[:, :f], gu[:, f:2 * f], form="clamped", limit=spec.shared_limit,
+                                          alpha=spec.alpha), w["shared_down"])
+        out = grouped_experts(x, w["gate_up"], w["down"], weights, ids, addend=shared if reduce else None,
+                              activation="clamped", gated=True, limit=spec.limit, alpha=spec.alpha, reduce=reduce)
+        return out if reduce else ExpertTerms(out, shared)
+    if not reduce:
+        raise ValueError("only the clamped experts hand out their terms")
     if spec.gated:
         # gated experts: [gate | up] stacked per expert; the shared expert's [gate | up | token-gate row] is one product
         if spec.shared_ff:
@@ -466,7 +559,8 @@ def moe_feed_forward(spec: MoeMlpSpec, w: dict[str, torch.Tensor], x: torch.Tens
 
 MIXERS = {"mamba2": mamba2_mixer, "attention": sink_attention_mixer, "latent_attention": latent_attention_mixer,
           "mingru": min_gru_mixer, "rglru": rg_lru_mixer, "parallel": side_by_side_mixer,
-          "forget_gate": forget_gate_mixer, "window_delta": window_delta_mixer}
+          "forget_gate": forget_gate_mixer, "window_delta": window_delta_mixer,
+          "window_attention": window_attention_mixer, "mlstm": mlstm_mixer}
 FEED_FORWARDS = {"dense": dense_feed_forward, "moe": moe_feed_forward}
 
 
@@ -485,6 +579,8 @@ class LayeredDecoder:
         design soft-caps its logits)."""
         cfg, eps, off, kind = self.cfg, self.cfg.rms_norm_eps, self.norm_offset, self.cfg.norm_kind
         ctx = StepContext(batch, kv_buffer, table, states)
+        if cfg.streams:
+            return self._forward_streams(tokens, ctx, want_rows)
         if cfg.single_norm:
             return self._forward_single_norm(tokens, ctx, want_rows)
         if cfg.parallel_block:
@@ -518,7 +614,11 @@ class LayeredDecoder:
 
     def _head(self, resid: torch.Tensor, want_rows: torch.Tensor | None) -> torch.Tensor:
         cfg = self.cfg
-        hidden = rmsnorm_from_f32(resid, self.w.final_norm, cfg.rms_norm_eps, self.norm_offset, want_rows, cfg.norm_kind)
+        return self._logits(rmsnorm_from_f32(resid, self.w.final_norm, cfg.rms_norm_eps, self.norm_offset, want_rows,
+                                             cfg.norm_kind))
+
+    def _logits(self, hidden: torch.Tensor) -> torch.Tensor:
+        cfg = self.cfg
         logits = linear(hidden, self.w.head)
         if cfg.logit_softcap or cfg.logit_scale != 1.0:
             return softcap_to_f32(logits, cfg.logit_softcap, cfg.logit_scale)
@@ -546,6 +646,53 @@ class LayeredDecoder:
         if want_rows is not None and want_rows.numel() == 0:
             return torch.empty((0, cfg.vocab_size), dtype=torch.float32, device=tokens.device)
         return self._head(resid, want_rows)
+
+    def _forward_streams(self, tokens: torch.Tensor, ctx: StepContext, want_rows: torch.Tensor | None) -> torch.Tensor:
+        """A residual of several fp32 streams.  Between two sublayers ONE kernel gates the finished sublayer's result (and
+        sums its expert terms), writes all streams, reads the next sublayer's input and norms it; in steps of single
+        tokens it also runs the input convolution.  The last such kernel reads the wanted rows only, through the final
+        norm, and writes nothing back."""
+        cfg, w, eps, b = self.cfg, self.w, self.cfg.rms_norm_eps, ctx.batch
+        if cfg.norm_kind != "rms" or self.norm_offset != 0.0 or not cfg.embed_norm or not cfg.layers:
+            raise ValueError("stream designs use plain RMS norms, a normed embedding and at least one layer")
+        subs = [(li, sub) for li, spec in enumerate(cfg.layers) for sub in range(1 if spec.mlp is None else 2)]
+
+        def conv_of(at: int):
+            if not cfg.input_conv or at == len(subs) or b.num_portions:
+                return None
+            li, sub = subs[at]
+            return w.layers[li].subs[sub]["conv"], ctx.states.input_tail[(li, sub)], b.seq_ctx, b.seq_slot
+
+        first = w.layers[0].subs[0]
+        x, h, hc = stream_embed(tokens, w.embed, w.embed_norm, cfg.streams, first["in"], first["norm"], eps, conv_of(0))
+        for at, (li, sub) in enumerate(subs):
+            spec, lw, sw = cfg.layers[li], w.layers[li], w.layers[li].subs[sub]
+            gate = linear(h, sw["gate"]) if cfg.sublayer_gate else None
+            if cfg.input_conv and hc is None:
+                hc = causal_conv_silu(h, 0, cfg.hidden_size, sw["conv"], None, ctx.states.input_tail[(li, sub)], b.seq_start,
+                                      b.seq_ctx, b.seq_slot, activation=False, residual=True)
+            inner = h if hc is None else hc
+            if sub == 0:
+                y = MIXERS[spec.kind](li, spec.mixer, lw.mix, inner, ctx, eps)
+            else:
+                y = FEED_FORWARDS[spec.mlp.kind](spec.mlp, lw.mlp, inner, reduce=False)
+            y, addend = (y.terms, y.addend) if isinstance(y, ExpertTerms) else (y, None)
+            write = dict(addend=addend, gate=gate, gate_bias=sw.get("gate_b"))
+            if at + 1 < len(subs):
+                nli, nsub = subs[at + 1]
+                nw = w.layers[nli].subs[nsub]
+                h, hc = stream_mix(x, y, sw["coef"], nw["in"], nw["norm"], eps, conv=conv_of(at + 1), **write)
+            elif self.layer_trace is not None:
+                h, _ = stream_mix(x, y, sw["coef"], w.stream_ones, w.final_norm, eps, **write)
+                if want_rows is not None:
+                    h = h.index_select(0, want_rows.long())
+            elif want_rows is None or want_rows.numel():
+                h, _ = stream_mix(x, y, sw["coef"], w.stream_ones, w.final_norm, eps, rows=want_rows, **write)
+            if self.layer_trace is not None and (at + 1 == len(subs) or subs[at + 1][0] != li):
+                self.layer_trace.append(x.sum(1))
+        if want_rows is not None and want_rows.numel() == 0:
+            return torch.empty((0, cfg.vocab_size), dtype=torch.float32, device=tokens.device)
+        return self._logits(h)
 
     def _forward_parallel(self, tokens: torch.Tensor, ctx: StepContext, want_rows: torch.Tensor | None) -> torch.Tensor:
         """Parallel blocks over a stack of fp32 results: level 0 is the (normed) embedding, level i + 1 the result of
@@ -1189,3 +1336,184 @@ _GOFEZEN_SOURCES = ("gemm_dense", "gemm_simt", "gemm_rows_mma", "residual_stream
                     "gated_linear_attention", "rotary_heads", "attention_sink", "moe_routing", "elementwise")
 register(Architecture("Gofezen", parse_gofezen_config, map_gofezen_weights, LayeredDecoder, ragged_steps=True,
                       sources=_GOFEZEN_SOURCES))
+
+
+# ---------------------------------------------------------------------------------------------- Torutar plumbing #
+def _torutar_mixer(kind: str, m: dict):
+    rot = m.get("rot") or {}
+    mask = m.get("mask") or {}
+    if kind == "attention":
+        return "window_attention", WindowAttentionSpec(
+            heads=int(m["heads"]), kv_heads=int(m.get("kv_heads", m["heads"])), head_dim=int(m["dim"]),
+            v_head_dim=int(m.get("vdim", m["dim"])), scale=float(m["scale"]), window=int(mask.get("size", 0)),
+            keep_first=int(mask.get("keep_first", 0)), rot_dims=int(rot.get("dims", 0)),
+            rot_base=float(rot.get("base", 10000.0)), kv_from=m.get("kv_from"))
+    if kind == "latent_attention":
+        rot_dim = int(m.get("rot_dim", 0))
+        return kind, LatentAttentionSpec(
+            heads=int(m["heads"]), head_dim=int(m["dim"]), rot_dim=rot_dim, v_head_dim=int(m.get("vdim", m["dim"])),
+            q_rank=int(m["q_rank"]), kv_rank=int(m["kv_rank"]), scale=float(m["scale"]),
+            rot_dims=int(rot.get("dims", rot_dim)), rot_base=float(rot.get("base", 10000.0)), element_gate=True,
+            pairing="neighbours")
+    if kind == "mlstm":
+        return kind, MlstmSpec(heads=int(m["heads"]), head_dim=int(m["dim"]), v_head_dim=int(m.get("vdim", m["dim"])),
+                               gate_cap=float(m["gate_cap"]))
+    raise ValueError(f"unknown layer type {kind!r}")
+
+
+def _torutar_mlp(mlp: dict | None) -> MoeMlpSpec | None:
+    if mlp is None:
+        return None
+    if mlp.get("kind", "moe") != "moe":
+        raise ValueError(f"unknown feed-forward kind {mlp.get('kind')!r}")
+    r, shared = mlp["router"], mlp.get("shared") or {}
+    return MoeMlpSpec(experts=int(r["experts"]), top=int(r["top"]), ff=int(mlp["expert"]["ff"]),
+                      shared_ff=int(shared.get("ff", 0)), activation="clamped", gated=True, scores="softmax",
+                      scale=float(r.get("scale", 1.0)), limit=float(mlp["expert"]["limit"]),
+                      shared_limit=float(shared.get("limit", 0.0)))
+
+
+def parse_torutar_config(raw: dict) -> LayeredConfig:
+    layers = []
+    for entry in raw["layers"]:
+        key, mixer = _torutar_mixer(entry["type"], entry["mixer"])
+        layers.append(LayerSpec(key, mixer, _torutar_mlp(entry.get("mlp"))))
+    return LayeredConfig(name=raw.get("architecture", "Torutar"), hidden_size=int(raw["width"]),
+                         vocab_size=int(raw["vocab"]), max_seq_len=0, rms_norm_eps=float(raw["norm"]["eps"]),
+                         layers=tuple(layers), norm_weight_offset=0.0, learned_positions=False, embed_norm=True,
+                         logit_scale=float(raw.get("logit_scale", 1.0)), streams=int(raw["streams"]),
+                         input_conv=int(raw["canon"]["taps"]), sublayer_gate=True)
+
+
+def _stack_aligned(parts: list[torch.Tensor]) -> torch.Tensor:
+    """Row-concatenation with every part starting on a multiple of 8 rows (``aligned_columns``)."""
+    return torch.cat([_pad_rows(p, 8) for p in parts], dim=0).contiguous()
+
+
+def map_torutar_weights(cfg: LayeredConfig, tensors: dict[str, torch.Tensor], device: str,
+                        dtype: torch.dtype) -> LayeredWeights:
+    """Checkpoint names -> the decoder's weights.  Every mixer's input projections are row-concatenated into one GEMM
+    weight (parts that a kernel reads with 16-byte accesses start on a multiple of 8 rows), with one bias vector where some
+    part has a bias; the latent key up-projection is stored transposed per head; experts are stacked with each expert's
+    gate and up rows interleaved; stream coefficients are fp32."""
+
+    def get(name: str, dt: torch.dtype = dtype) -> torch.Tensor:
+        if name not in tensors:
+            raise KeyError(f"checkpoint has no tensor {name!r}")
+        return tensors[name].to(device=device, dtype=dt).contiguous()
+
+    def zeros(n: int) -> torch.Tensor:
+        return torch.zeros(n, dtype=dtype, device=device)
+
+    out = LayeredWeights(embed=get("embed"), pos=None, final_norm=get("final.norm"), head=get("head"),
+                         embed_norm=get("embed.norm"),
+                         stream_ones=torch.ones(cfg.streams, dtype=torch.float32, device=device))
+    for i, spec in enumerate(cfg.layers):
+        p, m = f"l{i}.mix.", spec.mixer
+        if isinstance(m, WindowAttentionSpec):
+            names = ["q", "k", "v"] if m.kv_from is None else ["q"]
+            mix = {"in": _stack_aligned([torch.cat([get(p + n) for n in names], dim=0), get(p + "g")]),
+                   "in_b": _stack_aligned([torch.cat([get(f"{p}{n}.b") for n in names]), zeros(m.heads)]),
+                   "q_norm": get(p + "q.norm"), "sink": get(p + "sink"), "o": get(p + "o"), "o_b": get(p + "o.b")}
+            if m.kv_from is None:
+                mix["k_norm"] = get(p + "k.norm")
+        elif isinstance(m, LatentAttentionSpec):
+            uk = get(p + "uk").view(m.heads, m.head_dim, m.kv_rank)
+            mix = {"down": _pad_rows(torch.cat([get(p + "dq"), get(p + "dkv"), get(p + "g")], dim=0), 8).contiguous(),
+                   "q_norm": get(p + "dq.norm"), "kv_norm": get(p + "dkv.norm"), "uq": get(p + "uq"),
+                   "uk_t": uk.transpose(1, 2).contiguous(),
+                   "uv": get(p + "uv").view(m.heads, m.v_head_dim, m.kv_rank).contiguous(), "o": get(p + "o")}
+        else:
+            mix = {"in": _stack_aligned([get(p + n) for n in ("q", "k", "v", "g", "i", "f")]), "i_b": get(p + "i.b"),
+                   "f_b": get(p + "f.b"), "norm": get(p + "norm"), "o": get(p + "o")}
+        lw = LayeredLayerWeights(norm1=None, mix=mix, subs=[])
+        for q in range(1, 2 if spec.mlp is None else 3):
+            lw.subs.append({"norm": get(f"l{i}.norm{q}"), "in": get(f"l{i}.hc{q}.in", torch.float32),
+                            "coef": torch.cat([get(f"l{i}.hc{q}.out", torch.float32),
+                                               get(f"l{i}.hc{q}.mix", torch.float32).reshape(-1)]),
+                            "conv": get(f"l{i}.canon{q}"), "gate": get(f"l{i}.rg{q}"), "gate_b": get(f"l{i}.rg{q}.b")})
+        if spec.mlp is not None:
+            q, e = f"l{i}.mlp.", range(spec.mlp.experts)
+            lw.mlp = {"router": get(q + "router"),
+                      "gate_up": torch.stack([torch.stack([get(f"{q}e{j}.gate"), get(f"{q}e{j}.up")], dim=1).flatten(0, 1)
+                                              for j in e]).contiguous(),
+                      "down": torch.stack([get(f"{q}e{j}.down") for j in e]).contiguous()}
+            if q + "correction" in tensors:
+                lw.mlp["correction"] = get(q + "correction")
+            if spec.mlp.shared_ff:
+                lw.mlp["shared_gate_up"] = torch.cat([get(q + "shared.gate"), get(q + "shared.up")], dim=0).contiguous()
+                lw.mlp["shared_down"] = get(q + "shared.down")
+        out.layers.append(lw)
+    return out
+
+
+def torutar_tensor_shapes(cfg: LayeredConfig) -> dict[str, tuple[int, ...]]:
+    """Checkpoint tensor names and shapes of a configuration (random initialisation, shape checks)."""
+    w, s = cfg.hidden_size, cfg.streams
+    shapes: dict[str, tuple[int, ...]] = {"embed": (cfg.vocab_size, w), "embed.norm": (w,)}
+    for i, spec in enumerate(cfg.layers):
+        p, m = f"l{i}.mix.", spec.mixer
+        if isinstance(m, WindowAttentionSpec):
+            rows = {"q": m.heads * m.head_dim}
+            shapes[p + "q.norm"] = (m.head_dim,)
+            if m.kv_from is None:
+                rows.update({"k": m.kv_heads * m.head_dim, "v": m.kv_heads * m.v_head_dim})
+                shapes[p + "k.norm"] = (m.head_dim,)
+            for n, r in rows.items():
+                shapes.update({p + n: (r, w), f"{p}{n}.b": (r,)})
+            shapes.update({p + "sink": (m.heads,), p + "g": (m.heads, w), p + "o": (w, m.heads * m.v_head_dim), p + "o.b": (w,)})
+        elif isinstance(m, LatentAttentionSpec):
+            shapes.update({p + "dq": (m.q_rank, w), p + "dq.norm": (m.q_rank,),
+                           p + "uq": (m.heads * (m.head_dim + m.rot_dim), m.q_rank), p + "dkv": (m.kv_rank + m.rot_dim, w),
+                           p + "dkv.norm": (m.kv_rank,), p + "uk": (m.heads * m.head_dim, m.kv_rank),
+                           p + "uv": (m.heads * m.v_head_dim, m.kv_rank), p + "g": (m.heads * m.v_head_dim, w),
+                           p + "o": (w, m.heads * m.v_head_dim)})
+        else:
+            nq, nv = m.heads * m.head_dim, m.heads * m.v_head_dim
+            shapes.update({p + "q": (nq, w), p + "k": (nq, w), p + "v": (nv, w), p + "g": (nv, w), p + "o": (w, nv),
+                           p + "norm": (nv,), p + "i": (m.heads, w), p + "i.b": (m.heads,), p + "f": (m.heads, w),
+                           p + "f.b": (m.heads,)})
+        for q in range(1, 2 if spec.mlp is None else 3):
+            shapes.update({f"l{i}.norm{q}": (w,), f"l{i}.hc{q}.in": (s,), f"l{i}.hc{q}.out": (s,), f"l{i}.hc{q}.mix": (s, s),
+                           f"l{i}.canon{q}": (w, cfg.input_conv), f"l{i}.rg{q}": (w, w), f"l{i}.rg{q}.b": (w,)})
+        if spec.mlp is not None:
+            q = f"l{i}.mlp."
+            for e in [*(f"e{j}" for j in range(spec.mlp.experts)), *(["shared"] if spec.mlp.shared_ff else [])]:
+                f = spec.mlp.shared_ff if e == "shared" else spec.mlp.ff
+                shapes.update({f"{q}{e}.gate": (f, w), f"{q}{e}.up": (f, w), f"{q}{e}.down": (w, f)})
+            shapes.update({q + "router": (spec.mlp.experts, w), q + "correction": (spec.mlp.experts,)})
+    shapes.update({"final.norm": (w,), "head": (cfg.vocab_size, w)})
+    return shapes
+
+
+def random_torutar_tensors(cfg: LayeredConfig, seed: int = 0) -> dict[str, torch.Tensor]:
+    """Seeded random bf16 tensors with checkpoint names (benchmarks and tests; no trained checkpoints exist offline)."""
+    g = torch.Generator().manual_seed(seed)
+    out = {}
+    for name, shape in torutar_tensor_shapes(cfg).items():
+        leaf = name.rsplit(".", 1)[-1]
+        if leaf in ("canon1", "canon2"):
+            t = 0.3 * torch.randn(shape, generator=g)
+        elif leaf == "mix":                                   # mostly the stream itself, some of every other one
+            t = 0.1 * torch.randn(shape, generator=g) + 0.9 * torch.eye(shape[0])
+        elif leaf in ("in", "out"):
+            t = (1.0 if leaf == "out" else 1.0 / shape[0]) + 0.1 * torch.randn(shape, generator=g)
+        elif len(shape) == 2:
+            t = torch.randn(shape, generator=g) / (shape[1] ** 0.5)
+        elif leaf == "correction":
+            t = 0.02 * torch.randn(shape, generator=g)
+        elif leaf == "sink" or name.endswith(("q.b", "k.b", "v.b", "o.b", "i.b", "rg1.b", "rg2.b")):
+            t = 0.3 * torch.randn(shape, generator=g)
+        elif name.endswith("f.b"):                            # forget gates that mostly keep
+            t = 3.0 + 0.5 * torch.randn(shape, generator=g)
+        else:                                                 # norm weights
+            t = 1.0 + 0.1 * torch.randn(shape, generator=g)
+        out[name] = t.to(torch.bfloat16)
+    return out
+
+
+_TORUTAR_SOURCES = ("gemm_dense", "gemm_simt", "gemm_rows_mma", "residual_stream", "hyper_stream", "ssm_scan", "mlstm",
+                    "gated_linear_attention", "rotary_heads", "latent_attention", "attention_sink", "moe_routing",
+                    "elementwise")
+register(Architecture("Torutar", parse_torutar_config, map_torutar_weights, LayeredDecoder, ragged_steps=True,
+                      sources=_TORUTAR_SOURCES))

@@ -156,10 +156,13 @@ class LatentAttentionSpec:
     rot_base: float = 10000.0
     window: int = 0
     out_gate: bool = True
+    element_gate: bool = False                         # out_gate has one number per output element instead of per head
+    pairing: str = "halves"                            # rotary pairs: i, i + rot_dims / 2; "neighbours": 2i, 2i + 1
 
     def validate(self) -> None:
         if min(self.heads, self.head_dim, self.v_head_dim, self.q_rank, self.kv_rank) < 1 or self.rot_dim < 0 or \
-                self.rot_dims % 2 or not 0 <= self.rot_dims <= self.rot_dim or self.window < 0 or self.kv_rank > 256:
+                self.rot_dims % 2 or not 0 <= self.rot_dims <= self.rot_dim or self.window < 0 or self.kv_rank > 256 or \
+                self.pairing not in ("neighbours", "halves"):
             raise ValueError(f"unsupported latent attention geometry: {self}")
 
     @property
@@ -406,6 +409,61 @@ class WindowDeltaPairSpec:
 
 
 @dataclass(frozen=True)
+class WindowAttentionSpec:
+    """Softmax attention with biased projections, a per-head RMS norm of q and k (one ``[head_dim]`` weight each), rotary
+    positions on the first ``rot_dims`` entries (``pairing`` as in ``BlockAttentionSpec``), values divided by their root
+    mean square per head (``v_norm``), a sliding ``window`` (0: plain causal) in front of which the sequence's first
+    ``keep_first`` positions stay visible, a learned per-head sink in the softmax denominator and one logistic gate per
+    head on the output.  ``kv_from``: the layer whose cached keys and values this one reads (it has none of its own)."""
+
+    heads: int
+    kv_heads: int
+    head_dim: int
+    v_head_dim: int
+    scale: float
+    window: int = 0
+    keep_first: int = 0
+    rot_dims: int = 0
+    rot_base: float = 10000.0
+    pairing: str = "halves"
+    v_norm: bool = True
+    head_gate: bool = True
+    kv_from: int | None = None
+
+    @property
+    def cache_row_width(self) -> int:                  # all K heads, then all V heads, padded to 16-byte vectors
+        return -(-self.kv_heads * (self.head_dim + self.v_head_dim) // 8) * 8
+
+    def validate(self) -> None:
+        if min(self.heads, self.kv_heads, self.head_dim, self.v_head_dim) < 1 or self.heads % self.kv_heads or \
+                self.v_head_dim > 256 or self.window < 0 or self.keep_first < 0 or self.rot_dims % 2 or \
+                not 0 <= self.rot_dims <= self.head_dim or self.pairing not in ("neighbours", "halves"):
+            raise ValueError(f"unsupported attention geometry: {self}")
+
+
+@dataclass(frozen=True)
+class MlstmSpec:
+    """Matrix memory with exponential gates: per head an fp32 memory ``head_dim x v_head_dim``, a normaliser ``head_dim``
+    and a running log scale; input and forget gate logits are bounded by ``gate_cap`` (``cap tanh(. / cap)``; 0: not);
+    per-head RMS norm (weight ``[heads * v_head_dim]``), element-wise logistic gate, out-projection."""
+
+    heads: int
+    head_dim: int
+    v_head_dim: int
+    gate_cap: float = 0.0
+
+    @property
+    def state_shape(self) -> tuple[int, ...]:          # per head [memory | normaliser | log scale], padded to 16 bytes
+        return (self.heads, -(-(self.head_dim * self.v_head_dim + self.head_dim + 1) // 4) * 4)
+
+    conv_tail_shape = None
+
+    def validate(self) -> None:
+        if min(self.heads, self.head_dim, self.v_head_dim) < 1 or self.head_dim > 256:
+            raise ValueError(f"unsupported matrix-memory geometry: {self}")
+
+
+@dataclass(frozen=True)
 class DenseMlpSpec:
     ff: int
     activation: str = "relu2"                          # "relu2" | "gelu" | "gelu_tanh"; gated: "silu"
@@ -420,7 +478,10 @@ class MoeMlpSpec:
     neighbouring experts compete with the sum of their two best choice scores and only the ``keep`` best groups are
     eligible; the ``top`` winners' weights are their scores over the winners' sum, or (``renormalize=False``) the
     scores themselves.  ``weight_on_input``: an expert sees the token TIMES its weight instead of having its output
-    weighted.  ``shared_gate``: the shared expert's output is scaled by one logistic number per token."""
+    weighted.  ``shared_gate``: the shared expert's output is scaled by one logistic number per token.
+    ``scores="softmax"``: the scores are the softmax over all experts.  ``scale`` multiplies the weights.
+    ``activation="clamped"`` (gated): ``g' sigmoid(alpha g') (u' + 1)`` with ``g' = min(g, limit)`` and
+    ``u' = clamp(u, -limit, limit)``; the shared expert's bound is ``shared_limit``."""
 
     experts: int
     top: int
@@ -434,6 +495,11 @@ class MoeMlpSpec:
     renormalize: bool = True
     weight_on_input: bool = False
     shared_gate: bool = False
+    scores: str = "sigmoid"
+    scale: float = 1.0
+    limit: float = 0.0
+    shared_limit: float = 0.0
+    alpha: float = 1.702
 
     def validate(self) -> None:
         if self.experts < 1 or not 1 <= self.top <= self.experts or self.groups < 1 or self.experts % self.groups or \
@@ -444,7 +510,7 @@ class MoeMlpSpec:
 @dataclass(frozen=True)
 class LayerSpec:
     kind: str                                          # key of executor.layered_decoder.MIXERS
-    mixer: "Mamba2Spec | SinkAttentionSpec | LatentAttentionSpec | MinGruSpec | RgLruSpec | SideBySideSpec"
+    mixer: "Mamba2Spec | SinkAttentionSpec | LatentAttentionSpec | MinGruSpec | RgLruSpec | SideBySideSpec | WindowAttentionSpec | MlstmSpec"
     mlp: DenseMlpSpec | MoeMlpSpec | None = None
     weights_of: int | None = None                      # the layer whose tensors this one uses (cache / state are its own)
 
@@ -475,6 +541,13 @@ class LayeredConfig:
     # single_norm: a parallel block with ONE input norm that both sublayers read, x <- x + mixer(h) + ff(h), h = norm1(x)
     single_norm: bool = False
     logit_scale: float = 1.0                           # the head's output times this, before the soft cap
+    # streams > 0: the residual is kept as that many streams; a sublayer reads a weighted sum of them and writes all of
+    # them (hyper-connections).  input_conv > 0: what every sublayer reads, h, becomes h + a causal convolution of it with
+    # that many taps.  sublayer_gate: a sublayer's result is multiplied by sigmoid(W h + b) element-wise, h before the
+    # convolution
+    streams: int = 0
+    input_conv: int = 0
+    sublayer_gate: bool = False
 
     @property
     def num_layers(self) -> int:
@@ -482,6 +555,10 @@ class LayeredConfig:
 
     def attention_layers(self) -> list[int]:
         """Layers that keep rows in the KV pool (their mixer spec names the row width)."""
+        return [i for i in self.cache_readers() if getattr(self.layers[i].mixer, "kv_from", None) is None]
+
+    def cache_readers(self) -> list[int]:
+        """Layers whose mixer reads pool rows: their own, or those of the layer it names (``kv_from``)."""
         return [i for i, l in enumerate(self.layers) if hasattr(l.mixer, "cache_row_width")]
 
     def recurrent_layers(self) -> list[int]:
@@ -499,6 +576,13 @@ class LayeredConfig:
                     raise ValueError(f"layer {i} shares the weights of layer {j}, which has none of its own")
                 if (self.layers[j].kind, self.layers[j].mixer, self.layers[j].mlp) != (l.kind, l.mixer, l.mlp):
                     raise ValueError(f"layer {i} shares the weights of layer {j} but differs from it")
+            j = getattr(l.mixer, "kv_from", None)
+            if j is not None:
+                own = self.layers[j].mixer if 0 <= j < i else None
+                if not isinstance(own, WindowAttentionSpec) or own.kv_from is not None or \
+                        (own.kv_heads, own.head_dim, own.v_head_dim) != (l.mixer.kv_heads, l.mixer.head_dim, l.mixer.v_head_dim):
+                    raise ValueError(f"layer {i} reads the cache of layer {j}, which is no earlier attention layer of its "
+                                     "key and value sizes with a cache of its own")
         shared = {l.mixer.kv_heads * l.mixer.v_head_dim for l in self.layers
                   if isinstance(l.mixer, SinkAttentionSpec) and l.mixer.v_mix}
         if len(shared) > 1:

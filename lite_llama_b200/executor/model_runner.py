@@ -245,7 +245,7 @@ class RequestState:
         self.slot = slot
         self.num_cached = 0
         self.rows: list[int] = []          # the pool row of every position so far (released ones keep their entry)
-        self.released = 0                  # positions [0, released) have given their rows back (sliding windows)
+        self.released = 0                  # positions [keep_first, released) have given their rows back (sliding windows)
 
 
 class ModelRunner:
@@ -298,11 +298,14 @@ class ModelRunner:
         self.kv_cache_manager = KVCacheManager(len(attn), 0, 0, max_tokens, dtype=self.dtype, device=self.device,
                                                row_widths=widths)
         self.kv_buffer_of = dict(zip(attn, self.kv_cache_manager.gpu_kv_buffer))
-        # when EVERY cached layer has a sliding window, positions that no later token can see give their rows back
-        # while the request is still running: the longest window, plus one 64-key attention tile of slack (the tiled
-        # kernel starts its first key tile on a tile boundary below the window)
-        windows = [getattr(config.layers[i].mixer, "window", 0) for i in attn]
+        # when EVERY layer that reads the pool has a sliding window, positions that no later token can see give their
+        # rows back while the request is still running: the longest window, plus one 64-key attention tile of slack (the
+        # tiled kernel starts its first key tile on a tile boundary below the window); the first `keep_first` positions
+        # that some window keeps visible stay
+        readers = [config.layers[i].mixer for i in config.cache_readers()]
+        windows = [getattr(m, "window", 0) for m in readers]
         self.keep_positions = max(windows) - 1 + 64 if windows and min(windows) > 0 else 0
+        self.keep_first = max(getattr(m, "keep_first", 0) for m in readers) if self.keep_positions else 0
         # longest sequence = columns of the request table: the position table's length; without one, the pool's size, or
         # (rows are given back on the way) as far as the caller asks, 64k positions by default
         if config.max_seq_len > 0:
@@ -347,9 +350,9 @@ class ModelRunner:
         widths = tuple(w for w in widths if 1 <= w <= min(self.max_request_num, self.kv_cache_manager.max_num_tokens))
         caps = sorted({min(b, self.max_seq_len) for b in ctx_buckets} | {self.max_seq_len})
         if self.keep_positions:
-            # every cached layer has a window: a token sees at most `window` keys whatever its context, so all buckets
+            # every cached layer has a window: a token sees at most `window + keep_first` keys whatever its context, so all buckets
             # from the longest window up capture the same launches -- one graph (the longest bucket) serves them
-            longest = self.keep_positions + 1 - 64
+            longest = self.keep_positions + 1 - 64 + self.keep_first
             caps = [c for c in caps if c < longest] + [self.max_seq_len]
         try:
             for w in widths:
@@ -365,22 +368,26 @@ class ModelRunner:
     def close_request(self, req: RequestState) -> None:
         """Give the request's pool rows and its slot back."""
         if req.rows:
-            self.kv_cache_manager.release_rows_host(req.rows[req.released:])
+            self.kv_cache_manager.release_rows_host(self._held_rows(req))
             req.rows = []
         self.state_manager.release(req.slot)
         req.num_cached = req.released = 0
 
     def _release_unseen_rows(self, req: RequestState) -> None:
         """Sliding windows: the next token (position ``num_cached``) and all later ones see no position below
-        ``num_cached - keep_positions``; those rows go back to the pool now."""
+        ``num_cached - keep_positions`` except the first ``keep_first``; the rows between go back to the pool now."""
         if self.keep_positions:
             dead = req.num_cached - self.keep_positions
-            if dead > req.released:
-                self.kv_cache_manager.release_rows_host(req.rows[req.released:dead])
+            first = max(req.released, self.keep_first)
+            if dead > first:
+                self.kv_cache_manager.release_rows_host(req.rows[first:dead])
                 req.released = dead
 
+    def _held_rows(self, req: RequestState) -> list[int]:
+        return req.rows[:self.keep_first] + req.rows[req.released:] if req.released > self.keep_first else req.rows
+
     def rows_held(self, req: RequestState) -> int:
-        return len(req.rows) - req.released
+        return len(self._held_rows(req))
 
     def rows_needed(self, tokens: int) -> int:
         return tokens

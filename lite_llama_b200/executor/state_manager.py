@@ -2,7 +2,9 @@
 with the sequence: per recurrent layer one fp32 state tensor ``[slots, *spec.state_shape]`` (a state-space or
 linear-attention memory ``heads x state x head_dim``, or one value per channel of an element-wise recurrence) and,
 for mixers with a short convolution, its tail ``[slots, taps - 1, channels]`` (the last inputs, in the activation dtype;
-a mixer with several convolutions names one tail per convolution in ``spec.conv_tails``).
+a mixer with several convolutions names one tail per convolution in ``spec.conv_tails``).  Designs that convolve what
+every sublayer reads (``LayeredConfig.input_conv``) keep one more tail per sublayer of every layer: the last
+``input_conv - 1`` inputs ``[slots, input_conv - 1, hidden_size]``.
 
 A request holds one slot from admission to release; the same slot number indexes the request -> rows table of the
 KV pool (``ModelRunner.b_req_tokens_table``), as the reference's slot scheme does for attention
@@ -32,6 +34,12 @@ class RecurrentStateManager:
             if getattr(m, "conv_tails", None):
                 self.named_tail[i] = {name: torch.zeros((num_slots, *shape), dtype=dtype, device=device)
                                       for name, shape in m.conv_tails.items()}
+        self.input_tail: dict[tuple[int, int], torch.Tensor] = {}    # (layer, sublayer 0 mixer / 1 feed-forward)
+        if config.input_conv:
+            for i, layer in enumerate(config.layers):
+                for sub in range(1 if layer.mlp is None else 2):
+                    self.input_tail[(i, sub)] = torch.zeros((num_slots, max(config.input_conv - 1, 1), config.hidden_size),
+                                                            dtype=dtype, device=device)
         self._free = list(range(num_slots - 1, -1, -1))
         self._held: set[int] = set()
 
@@ -54,4 +62,5 @@ class RecurrentStateManager:
 
     def nbytes(self) -> int:
         named = [t for d in self.named_tail.values() for t in d.values()]
-        return sum(t.numel() * t.element_size() for t in [*self.ssm_state.values(), *self.conv_tail.values(), *named])
+        return sum(t.numel() * t.element_size() for t in [*self.ssm_state.values(), *self.conv_tail.values(), *named,
+                                                          *self.input_tail.values()])

@@ -9,6 +9,7 @@ import torch
 from ._common import check, dtype_code, float_code, index_width, lib, ptr, require_cuda, stream_handle
 
 _KIND_F16, _KIND_FP8, _KIND_INT8 = 0, 1, 2
+SCORES = {"sigmoid": 0, "softmax": 1}
 
 
 @torch.no_grad()
@@ -169,12 +170,13 @@ def route_topk(router_logits: torch.Tensor, top_k: int, renormalize: bool = True
 
 @torch.no_grad()
 def route_sigmoid_groups(x: torch.Tensor, router_w: torch.Tensor, bias: torch.Tensor | None, top_k: int,
-                         groups: int = 1, keep: int = 1, renormalize: bool = True):
+                         groups: int = 1, keep: int = 1, renormalize: bool = True, scores: str = "sigmoid",
+                         scale: float = 1.0):
     """Sigmoid router with a selection bias and group-limited choice (router product with fp32 results + one selection
     launch; a single launch for shapes no GEMM takes):
-    ``s = sigmoid(router_w @ x)`` in fp32; experts compete with ``s + bias``; they form ``groups`` runs of neighbours,
+    ``s = sigmoid(router_w @ x)`` (``scores="softmax"``: the softmax over all experts) in fp32; experts compete with ``s + bias``; they form ``groups`` runs of neighbours,
     a group scores the sum of its two best, only the ``keep`` best groups are eligible; the ``top_k`` winners' weights
-    are their ``s`` over the winners' sum (``renormalize=False``: their ``s`` as they are).  Returns ``(weights fp32 [T, k], ids int32 [T, k])``.  The reference's
+    are their ``s`` over the winners' sum (``renormalize=False``: their ``s`` as they are), times ``scale``.  Returns ``(weights fp32 [T, k], ids int32 [T, k])``.  The reference's
     router is a softmax over all experts (lite_llama/models/qwen3_moe.py:94-100, ``route_topk``)."""
     require_cuda(x, router_w, bias)
     if x.stride(-1) != 1:
@@ -199,22 +201,23 @@ def route_sigmoid_groups(x: torch.Tensor, router_w: torch.Tensor, bias: torch.Te
         check(L.b2l_linear_f32out_mma(logits.data_ptr(), x.data_ptr(), router_w.data_ptr(), tokens, e, k, x.stride(0), e,
                                       code, stream_handle()))
     check(L.b2l_moe_route_sigmoid_groups(w.data_ptr(), ids.data_ptr(), x.data_ptr(), x.stride(0), router_w.data_ptr(),
-                                         ptr(bias), ptr(logits), tokens, e, k, int(top_k), int(groups), int(keep), 1 if renormalize else 0, code,
-                                         stream_handle()))
+                                         ptr(bias), ptr(logits), tokens, e, k, int(top_k), int(groups), int(keep),
+                                         1 if renormalize else 0, SCORES[scores], float(scale), code, stream_handle()))
     return w, ids
 
 
 def _swiglu_into(mid: torch.Tensor, wide: torch.Tensor, ff: int, in_scale: torch.Tensor | None) -> None:
     """``mid = silu(s * wide[:, :ff]) * (s * wide[:, ff:])`` with the per-slot fp32 factor ``s`` (optional)."""
     check(lib().b2l_swiglu_scaled(mid.data_ptr(), mid.stride(0), wide.data_ptr(), wide.stride(0), wide[:, ff:].data_ptr(),
-                                  wide.stride(0), ptr(in_scale), None, 0, mid.shape[0], ff, float_code(mid, "mid"),
-                                  stream_handle()))
+                                  wide.stride(0), ptr(in_scale), None, 0, mid.shape[0], ff, 0, 0.0, 0.0,
+                                  float_code(mid, "mid"), stream_handle()))
 
 
 @torch.no_grad()
 def grouped_experts(x: torch.Tensor, w_up: torch.Tensor, w_down: torch.Tensor, weights: torch.Tensor,
                     ids: torch.Tensor, addend: torch.Tensor | None = None, activation: str = "gelu",
-                    gated: bool = False, weight_on_input: bool = False) -> torch.Tensor:
+                    gated: bool = False, weight_on_input: bool = False, limit: float = 0.0,
+                    alpha: float = 1.702, reduce: bool = True) -> torch.Tensor:
     """``sum_k weights[t, k] * W_down[e] act(W_up[e] x[t]) (+ addend[t])`` over each token's chosen experts
     ``e = ids[t, k]``: ungated two-matrix experts, ``w_up [E, ff, h]``, ``w_down [E, h, ff]``.  Slots are sorted by
     expert (``moe_align_block_size``), both products run grouped (``mma.sync`` tiles for aligned 16-bit operands, the
@@ -222,10 +225,15 @@ def grouped_experts(x: torch.Tensor, w_up: torch.Tensor, w_down: torch.Tensor, w
     in the second's.  ``gated`` (``activation="silu"``): ``w_up [E, 2 * ff, h]`` holds every expert's gate rows then its
     up rows, and the unit is ``W_down (silu(W_gate x) * W_up x)``; the activation is a kernel of its own between the
     products.  ``weight_on_input``: the expert sees ``weights[t, k] * x[t]`` and its output is not weighted; the factor
-    passes through the first (linear) product and is applied to its fp32-widened results.  The fp16 / fp8 gated experts
+    passes through the first (linear) product and is applied to its fp32-widened results.
+    ``activation="clamped"`` (gated): ``w_up`` interleaves every expert's rows (2i: gate i, 2i + 1: up i) and the unit
+    ``g' sigmoid(alpha g') (u' + 1)``, ``g' = min(g, limit)``, ``u' = clamp(u, -limit, limit)`` is formed from the fp32
+    sums in the first product's epilogue, so the two halves are never stored.  ``reduce=False``: the weighted outputs
+    of a token's experts are returned as ``[tokens, top_k, h]`` for a consumer that sums them itself.  The fp16 / fp8 gated experts
     of the reference's family are ``fused_moe``."""
     require_cuda(x, w_up, w_down, weights, ids, addend)
-    if (activation, gated) not in (("gelu", False), ("silu", True)) or (weight_on_input and not gated):
+    if (activation, gated) not in (("gelu", False), ("silu", True), ("clamped", True)) or \
+            (weight_on_input and (activation, gated) != ("silu", True)):
         raise ValueError(f"grouped_experts: unknown expert form {activation!r}, gated={gated}")
     if weights.dtype != torch.float32:
         raise ValueError("grouped_experts: routing weights are fp32")
@@ -240,11 +248,13 @@ def grouped_experts(x: torch.Tensor, w_up: torch.Tensor, w_down: torch.Tensor, w
     w_up, w_down = w_up.contiguous(), w_down.contiguous()
     slots = tokens * top_k
     mid = torch.empty((slots, ff), dtype=x.dtype, device=x.device)
-    wide = torch.empty((slots, up_rows), dtype=x.dtype, device=x.device) if gated else mid
+    fused = activation == "clamped"                 # the unit is formed in the first product's epilogue
+    wide = torch.empty((slots, up_rows), dtype=x.dtype, device=x.device) if gated and not fused else mid
     expanded = torch.empty((slots, hidden), dtype=x.dtype, device=x.device)
     flat_w = weights.reshape(-1).contiguous()
     down_w = None if weight_on_input else flat_w.data_ptr()
-    act = 0 if gated else 1
+    act = 2 if fused else (0 if gated else 1)
+    unit = (float(limit), float(alpha))
     # 16-bit operands with 16-byte aligned rows run on the tensor cores (blocks of 16, 64 or 128 slots by the expected
     # slots per expert), everything else on the CUDA cores; the result of a slot does not depend on the block size
     tensor = bool(L.b2l_rows_gemm_mma_ok(x.data_ptr(), w_up.data_ptr(), hidden, x.stride(0), 0, code)) and \
@@ -255,21 +265,23 @@ def grouped_experts(x: torch.Tensor, w_up: torch.Tensor, w_down: torch.Tensor, w
     common = (sorted_ids.data_ptr(), expert_ids.data_ptr(), num_post.data_ptr(), sorted_ids.numel(), slots)
 
     def between() -> None:
-        if gated:
+        if gated and not fused:
             _swiglu_into(mid, wide, ff, flat_w if weight_on_input else None)
 
     if tensor:
         check(L.b2l_moe_gemm_mma(wide.data_ptr(), x.data_ptr(), w_up.data_ptr(), None, *common, top_k, block, up_rows,
-                                 hidden, x.stride(0), wide.stride(0), act, code, stream_handle()))
+                                 hidden, x.stride(0), wide.stride(0), act, *unit, code, stream_handle()))
         between()
         check(L.b2l_moe_gemm_mma(expanded.data_ptr(), mid.data_ptr(), w_down.data_ptr(), down_w, *common, 1,
-                                 block, hidden, ff, mid.stride(0), expanded.stride(0), 0, code, stream_handle()))
+                                 block, hidden, ff, mid.stride(0), expanded.stride(0), 0, *unit, code, stream_handle()))
     else:
         check(L.b2l_moe_gemm_simt(wide.data_ptr(), x.data_ptr(), w_up.data_ptr(), None, *common, top_k, up_rows, hidden,
-                                  x.stride(0), wide.stride(0), act, code, stream_handle()))
+                                  x.stride(0), wide.stride(0), act, *unit, code, stream_handle()))
         between()
         check(L.b2l_moe_gemm_simt(expanded.data_ptr(), mid.data_ptr(), w_down.data_ptr(), down_w, *common, 1,
-                                  hidden, ff, mid.stride(0), expanded.stride(0), 0, code, stream_handle()))
+                                  hidden, ff, mid.stride(0), expanded.stride(0), 0, *unit, code, stream_handle()))
+    if not reduce:
+        return expanded.view(tokens, top_k, hidden)
     out = torch.empty((tokens, hidden), dtype=x.dtype, device=x.device)
     check(L.b2l_moe_sum(out.data_ptr(), expanded.data_ptr(), ptr(addend), tokens, hidden, top_k, code, stream_handle()))
     return out

@@ -5,8 +5,9 @@ from __future__ import annotations
 
 import torch
 
-from ._common import check, float_code, lib, ptr, require_cuda, stream_handle
+from ._common import check, counters, float_code, lib, ptr, require_cuda, stream_handle
 
+GATED_UNITS = {"silu": 0, "clamped": 1}
 GATED_LINEAR_MODES = {"forget_gate": 0, "delta_rule": 1}
 
 
@@ -40,20 +41,69 @@ def gated_linear_scan(mode: str, state: torch.Tensor, q: torch.Tensor, k: torch.
     return y
 
 
+MLSTM_CHUNK = 64
+
+
+def mlstm_head_floats(dim: int, vdim: int) -> int:
+    """Floats of one head's state block ``[S: dim x vdim | n: dim | m]``, padded to 16 bytes (the layout of
+    csrc/mlstm.cu; ``b2l_mlstm_head_floats``)."""
+    return -(-(dim * vdim + dim + 1) // 4) * 4
+
+
+@torch.no_grad()
+def mlstm(state: torch.Tensor, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, zi: torch.Tensor, zf: torch.Tensor,
+          bias_i: torch.Tensor, bias_f: torch.Tensor, batch, heads: int, dim: int, vdim: int, gate_cap: float,
+          q_scale: float) -> torch.Tensor:
+    """Matrix memory with exponential gates over a ragged step: ``y [tokens, heads * vdim]`` fp32; ``state [slots, heads,
+    mlstm_head_floats(dim, vdim)]`` fp32 advanced in place.  ``q``, ``k``, ``v`` and the gate logits ``zi``, ``zf
+    [tokens, heads]`` are column views of a projection; ``i = cap tanh((zi + bias_i) / cap)``,
+    ``f = logsigmoid(cap tanh((zf + bias_f) / cap))``, ``m' = max(f + m, i)``,
+    ``S <- e^(f + m - m') S + e^(i - m') k v^T``, ``n`` likewise,
+    ``y = S^T q / (max(|n . q|, e^(-m')) + 1e-6)`` with ``q`` times ``q_scale``.  Portions of 16-bit steps that bring at
+    least a quarter of a chunk run chunk by chunk on the tensor cores (``dim <= 128``), everything else token by token."""
+    require_cuda(state, q, k, v, zi, zf, bias_i, bias_f)
+    if state.dtype != torch.float32 or not state.is_contiguous() or state.shape[1:] != (heads, mlstm_head_floats(dim, vdim)):
+        raise ValueError("mlstm: the state is a contiguous fp32 [slots, heads, mlstm_head_floats] tensor")
+    for t in (q, k, v, zi, zf):
+        if t.stride(-1) != 1 or t.dtype != q.dtype:
+            raise ValueError("mlstm: the inputs are column views of one dtype")
+    if bias_i.dtype != q.dtype or bias_f.dtype != q.dtype:
+        raise ValueError("mlstm: gate biases in the activation dtype")
+    y = torch.empty((q.shape[0], heads * vdim), dtype=torch.float32, device=q.device)
+    cnt = counters(q.device)
+
+    def run(seq_list, count: int, chunked: int) -> None:
+        check(lib().b2l_mlstm(y.data_ptr(), state.data_ptr(), q.data_ptr(), q.stride(0), k.data_ptr(), k.stride(0),
+                              v.data_ptr(), v.stride(0), zi.data_ptr(), zi.stride(0), zf.data_ptr(), zf.stride(0),
+                              bias_i.data_ptr(), bias_f.data_ptr(), batch.seq_start.data_ptr(), batch.seq_ctx.data_ptr(),
+                              batch.seq_slot.data_ptr(), ptr(seq_list), count, heads, dim, vdim, float(q_scale),
+                              float(gate_cap), cnt.data_ptr(), cnt.numel(), chunked, float_code(q, "q"), stream_handle()))
+
+    if q.dtype != torch.float32 and dim <= 128 and batch.max_portion >= MLSTM_CHUNK // 4:
+        run(batch.portion_list, batch.num_portions, 1)
+        if batch.num_singles:
+            run(batch.single_list, batch.num_singles, 0)
+    else:
+        run(None, batch.num_seqs, 0)
+    return y
+
+
 @torch.no_grad()
 def head_norm_gate(y: torch.Tensor, weight: torch.Tensor, heads: int, eps: float,
-                   gate: torch.Tensor | None = None) -> torch.Tensor:
-    """``unit_rms(y[t, h, :]) * weight * silu(gate[t, h, :])`` per head (``gate=None``: no gate); ``y`` fp32
-    ``[tokens, heads * vdim]``, ``weight [vdim]`` shared by the heads, output in ``weight``'s dtype."""
+                   gate: torch.Tensor | None = None, gate_form: str = "silu") -> torch.Tensor:
+    """``unit_rms(y[t, h, :]) * weight * silu(gate[t, h, :])`` per head (``gate=None``: no gate; ``gate_form="sigmoid"``:
+    its sigmoid); ``y`` fp32 ``[tokens, heads * vdim]``, ``weight [vdim]`` shared by the heads or ``[heads * vdim]``,
+    output in ``weight``'s dtype."""
     require_cuda(y, weight, gate)
     rows, inner = y.shape
     vdim = inner // heads
-    if y.dtype != torch.float32 or not y.is_contiguous() or weight.numel() != vdim or heads * vdim != inner or \
-            (gate is not None and (gate.stride(-1) != 1 or gate.dtype != weight.dtype)):
+    if y.dtype != torch.float32 or not y.is_contiguous() or weight.numel() not in (vdim, inner) or heads * vdim != inner or \
+            gate_form not in ("silu", "sigmoid") or (gate is not None and (gate.stride(-1) != 1 or gate.dtype != weight.dtype)):
         raise ValueError("head_norm_gate: bad layout")
     out = torch.empty((rows, inner), dtype=weight.dtype, device=y.device)
     check(lib().b2l_head_norm_gate(out.data_ptr(), y.data_ptr(), ptr(gate), gate.stride(0) if gate is not None else 0,
-                                   weight.data_ptr(), rows, heads, vdim, float(eps), float_code(weight, "weight"),
+                                   weight.data_ptr(), rows, heads, vdim, float(eps), 1 if gate_form == "sigmoid" else 0,
+                                   1 if weight.numel() == inner and heads > 1 else 0, float_code(weight, "weight"),
                                    stream_handle()))
     return out
 
@@ -76,10 +126,12 @@ def head_mix(wide: torch.Tensor, mix: torch.Tensor, heads: int, kv_heads: int, p
 
 @torch.no_grad()
 def swiglu_scaled(gate: torch.Tensor, up: torch.Tensor, in_scale: torch.Tensor | None = None,
-                  out_logit: torch.Tensor | None = None) -> torch.Tensor:
+                  out_logit: torch.Tensor | None = None, form: str = "silu", limit: float = 0.0,
+                  alpha: float = 1.702) -> torch.Tensor:
     """``silu(s * gate) * (s * up) * sigmoid(z)`` with one fp32 factor ``s = in_scale[r]`` and one logit
     ``z = out_logit[r, 0]`` per row (both optional).  A factor on a gated unit's INPUT passes through its two linear
-    maps, so it is applied here, between the products and the activation."""
+    maps, so it is applied here, between the products and the activation.  ``form="clamped"``: the unit is
+    ``g' sigmoid(alpha g') (u' + 1)`` with ``g' = min(g, limit)``, ``u' = clamp(u, -limit, limit)`` instead."""
     require_cuda(gate, up, in_scale, out_logit)
     rows, n = gate.shape
     if up.shape != gate.shape or gate.stride(-1) != 1 or up.stride(-1) != 1 or up.dtype != gate.dtype or \
@@ -89,6 +141,6 @@ def swiglu_scaled(gate: torch.Tensor, up: torch.Tensor, in_scale: torch.Tensor |
     out = torch.empty((rows, n), dtype=gate.dtype, device=gate.device)
     check(lib().b2l_swiglu_scaled(out.data_ptr(), out.stride(0), gate.data_ptr(), gate.stride(0), up.data_ptr(),
                                   up.stride(0), ptr(in_scale), ptr(out_logit),
-                                  out_logit.stride(0) if out_logit is not None else 0, rows, n, float_code(gate, "gate"),
-                                  stream_handle()))
+                                  out_logit.stride(0) if out_logit is not None else 0, rows, n, GATED_UNITS[form],
+                                  float(limit), float(alpha), float_code(gate, "gate"), stream_handle()))
     return out

@@ -53,19 +53,23 @@ def rope_table_freqs(positions: torch.Tensor, freqs: torch.Tensor, magnitude: fl
 
 
 @torch.no_grad()
-def head_norm_rope_prepare(qkv: torch.Tensor, kv_pool: torch.Tensor, kv_rows: torch.Tensor,
+def head_norm_rope_prepare(qkv: torch.Tensor, kv_pool: torch.Tensor | None, kv_rows: torch.Tensor,
                            cos_sin: torch.Tensor | None, q_norm: torch.Tensor | None, k_norm: torch.Tensor | None,
                            heads: int, kv_heads: int, head_dim: int, v_head_dim: int, rot_dims: int, eps: float,
-                           pairing: str = "neighbours") -> None:
+                           pairing: str = "neighbours", v_norm: bool = False) -> None:
     """Per token of ``qkv [T, heads*head_dim + kv_heads*(head_dim + v_head_dim)]``: per-head RMS norm of q and k (one
     ``[head_dim]`` weight each), rotation of the first ``rot_dims`` entries of every head by the token's row of
-    ``cos_sin``, q in place, ``[k | v]`` into pool row ``kv_rows[t]``."""
+    ``cos_sin``, q in place, ``[k | v]`` into pool row ``kv_rows[t]`` (``v_norm``: every v head divided by its root mean
+    square first).  ``kv_heads = 0``: q alone, nothing is cached (``kv_pool`` may be ``None``)."""
     require_cuda(qkv, kv_pool, kv_rows, cos_sin, q_norm, k_norm)
-    if qkv.stride(-1) != 1 or kv_pool.stride(-1) != 1 or kv_pool.shape[1] < kv_heads * (head_dim + v_head_dim):
+    if qkv.stride(-1) != 1 or (kv_pool is None and kv_heads) or (kv_pool is not None and (
+            kv_pool.stride(-1) != 1 or kv_pool.shape[1] < kv_heads * (head_dim + v_head_dim))):
         raise ValueError("head_norm_rope_prepare: bad layout")
     if cos_sin is not None and (cos_sin.dtype != torch.float32 or cos_sin.shape[1] != rot_dims or not cos_sin.is_contiguous()):
         raise ValueError("head_norm_rope_prepare: cos_sin is fp32 [T, rot_dims]")
-    check(lib().b2l_head_norm_rope_prepare(qkv.data_ptr(), qkv.stride(0), kv_pool.data_ptr(), kv_pool.stride(0),
+    check(lib().b2l_head_norm_rope_prepare(qkv.data_ptr(), qkv.stride(0), ptr(kv_pool),
+                                           kv_pool.stride(0) if kv_pool is not None else 0,
                                            kv_rows.data_ptr(), ptr(cos_sin), ptr(q_norm), ptr(k_norm), qkv.shape[0],
                                            heads, kv_heads, head_dim, v_head_dim, rot_dims if cos_sin is not None else 0,
-                                           PAIRINGS[pairing], float(eps), float_code(qkv, "qkv"), stream_handle()))
+                                           PAIRINGS[pairing], 1 if v_norm else 0, float(eps), float_code(qkv, "qkv"),
+                                           stream_handle()))

@@ -8,19 +8,19 @@ from ._common import check, float_code, lib, ptr, require_cuda, stream_handle
 
 
 @torch.no_grad()
-def causal_conv_silu(proj: torch.Tensor, col: int, channels: int, weight: torch.Tensor, bias: torch.Tensor,
-                     tail: torch.Tensor, seq_start: torch.Tensor, seq_ctx: torch.Tensor, seq_slot: torch.Tensor,
-                     activation: bool = True):
+def causal_conv_silu(proj: torch.Tensor, col: int, channels: int, weight: torch.Tensor, bias: torch.Tensor | None,
+                     tail: torch.Tensor | None, seq_start: torch.Tensor, seq_ctx: torch.Tensor, seq_slot: torch.Tensor,
+                     activation: bool = True, residual: bool = False):
     """``silu(conv(proj[:, col:col+channels]))`` per channel over a ragged step (``activation=False``: the plain
-    convolution); ``tail [slots, taps-1, channels]`` supplies the inputs of earlier steps and is advanced in place."""
+    convolution; ``residual``: the input itself is added first); ``tail [slots, taps-1, channels]`` supplies the inputs of earlier steps and is advanced in place."""
     require_cuda(proj, weight, bias, tail, seq_start, seq_ctx, seq_slot)
     tokens = proj.shape[0]
     taps = weight.shape[1]
     out = torch.empty((tokens, channels), dtype=proj.dtype, device=proj.device)
     view = proj[:, col:col + channels]
-    check(lib().b2l_causal_conv_silu(out.data_ptr(), view.data_ptr(), proj.stride(0), weight.data_ptr(), bias.data_ptr(),
+    check(lib().b2l_causal_conv_silu(out.data_ptr(), view.data_ptr(), proj.stride(0), weight.data_ptr(), ptr(bias),
                                      ptr(tail), seq_start.data_ptr(), seq_ctx.data_ptr(), seq_slot.data_ptr(),
-                                     seq_ctx.numel(), tokens, channels, taps, 1 if activation else 0,
+                                     seq_ctx.numel(), tokens, channels, taps, 1 if activation else 0, 1 if residual else 0,
                                      float_code(proj, "proj"), stream_handle()))
     return out
 
