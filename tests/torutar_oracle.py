@@ -228,3 +228,116 @@ def forward(config: dict, tensors: dict, tokens, return_layers: bool = False):
     z = np.stack([unit_rms(r, eps) for r in x.sum(0)]) * fn @ f64(tensors["head"]).T
     z = z * float(config.get("logit_scale", 1.0))
     return (z, layers) if return_layers else z
+
+
+# ------------------------------------------------------------------------------------------- test model builders #
+def attention_layer(heads=3, kv_heads=1, dim=6, vdim=5, size=9, keep_first=2, rot=4, base=1000.0, scale=0.4, kv_from=None,
+                    mlp="moe") -> dict:
+    m = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": scale}
+    if size:
+        m["mask"] = {"size": size, "keep_first": keep_first}
+    if rot:
+        m["rot"] = {"dims": rot, "base": base}
+    if kv_from is not None:
+        m["kv_from"] = kv_from
+    return {"type": "attention", "mixer": m, "mlp": moe_mlp() if mlp == "moe" else mlp}
+
+
+def latent_layer(heads=2, dim=5, rot_dim=4, vdim=3, q_rank=7, kv_rank=6, base=500.0, scale=0.5, mlp="moe") -> dict:
+    return {"type": "latent_attention", "mixer": {"heads": heads, "dim": dim, "rot_dim": rot_dim, "vdim": vdim,
+                                                  "q_rank": q_rank, "kv_rank": kv_rank, "scale": scale,
+                                                  "rot": {"dims": rot_dim, "base": base}},
+            "mlp": moe_mlp() if mlp == "moe" else mlp}
+
+
+def mlstm_layer(heads=2, dim=4, vdim=6, gate_cap=6.0, mlp="moe") -> dict:
+    return {"type": "mlstm", "mixer": {"heads": heads, "dim": dim, "vdim": vdim, "gate_cap": gate_cap},
+            "mlp": moe_mlp() if mlp == "moe" else mlp}
+
+
+def moe_mlp(experts=5, top=2, ff=6, limit=0.9, scale=1.7, shared_ff=7, shared_limit=0.6) -> dict:
+    out = {"kind": "moe", "expert": {"ff": ff, "limit": limit}, "router": {"experts": experts, "top": top, "scale": scale}}
+    if shared_ff:
+        out["shared"] = {"ff": shared_ff, "limit": shared_limit}
+    return out
+
+
+def make_config(layers, width=24, vocab=50, eps=1e-5, streams=2, taps=4, logit_scale=0.7) -> dict:
+    return {"architecture": "Torutar", "width": width, "vocab": vocab, "norm": {"eps": eps}, "streams": streams,
+            "canon": {"taps": taps}, "logit_scale": logit_scale, "layers": list(layers)}
+
+
+def tensor_shapes(config: dict) -> dict:
+    w, s, taps = config["width"], config["streams"], config["canon"]["taps"]
+    out = {"embed": (config["vocab"], w), "embed.norm": (w,), "final.norm": (w,), "head": (config["vocab"], w)}
+    for i, layer in enumerate(config["layers"]):
+        p, m = f"l{i}.mix.", layer["mixer"]
+        if layer["type"] == "attention":
+            parts = {"q": m["heads"] * m["dim"]}
+            if m.get("kv_from") is None:
+                parts.update({"k": m["kv_heads"] * m["dim"], "v": m["kv_heads"] * m["vdim"]})
+                out[p + "k.norm"] = (m["dim"],)
+            for name, rows in parts.items():
+                out.update({p + name: (rows, w), f"{p}{name}.b": (rows,)})
+            out.update({p + "q.norm": (m["dim"],), p + "sink": (m["heads"],), p + "g": (m["heads"], w),
+                        p + "o": (w, m["heads"] * m["vdim"]), p + "o.b": (w,)})
+        elif layer["type"] == "latent_attention":
+            H, D, R, V, K, Q = (m[k] for k in ("heads", "dim", "rot_dim", "vdim", "kv_rank", "q_rank"))
+            out.update({p + "dq": (Q, w), p + "dq.norm": (Q,), p + "uq": (H * (D + R), Q), p + "dkv": (K + R, w),
+                        p + "dkv.norm": (K,), p + "uk": (H * D, K), p + "uv": (H * V, K), p + "g": (H * V, w),
+                        p + "o": (w, H * V)})
+        else:
+            H, D, V = m["heads"], m["dim"], m["vdim"]
+            out.update({p + "q": (H * D, w), p + "k": (H * D, w), p + "v": (H * V, w), p + "g": (H * V, w),
+                        p + "o": (w, H * V), p + "norm": (H * V,), p + "i": (H, w), p + "i.b": (H,), p + "f": (H, w),
+                        p + "f.b": (H,)})
+        for q in (1,) if layer.get("mlp") is None else (1, 2):
+            a = f"l{i}."
+            out.update({f"{a}norm{q}": (w,), f"{a}canon{q}": (w, taps), f"{a}rg{q}": (w, w), f"{a}rg{q}.b": (w,),
+                        f"{a}hc{q}.in": (s,), f"{a}hc{q}.out": (s,), f"{a}hc{q}.mix": (s, s)})
+        mlp, q = layer.get("mlp"), f"l{i}.mlp."
+        if mlp is None:
+            continue
+        names = [f"e{e}" for e in range(mlp["router"]["experts"])] + (["shared"] if mlp.get("shared") else [])
+        for name in names:
+            f = mlp["shared"]["ff"] if name == "shared" else mlp["expert"]["ff"]
+            out.update({f"{q}{name}.gate": (f, w), f"{q}{name}.up": (f, w), f"{q}{name}.down": (w, f)})
+        out.update({q + "router": (mlp["router"]["experts"], w), q + "correction": (mlp["router"]["experts"],)})
+    return out
+
+
+def random_model(config: dict, seed: int = 0, spread: float = 1.0) -> dict:
+    """Random tensors (torch, fp32 holding bf16-exact values) with checkpoint names; ``spread`` widens the head so
+    that greedy choices are decided by more than rounding."""
+    import torch
+
+    g = torch.Generator().manual_seed(seed)
+    out = {}
+    for name, shape in tensor_shapes(config).items():
+        leaf = name.rsplit(".", 1)[-1]
+        if leaf in ("canon1", "canon2"):
+            t = 0.4 * torch.randn(shape, generator=g)
+        elif leaf == "mix":
+            t = 0.3 * torch.randn(shape, generator=g) + 0.7 * torch.eye(shape[0])
+        elif leaf in ("in", "out"):
+            t = 0.6 + 0.5 * torch.randn(shape, generator=g)
+        elif name == "head":
+            t = spread * torch.randn(shape, generator=g) / shape[1] ** 0.5
+        elif leaf == "router":
+            t = 3.0 * torch.randn(shape, generator=g) / shape[1] ** 0.5
+        elif leaf in ("gate", "up"):                         # some units reach their bound
+            t = 1.5 * torch.randn(shape, generator=g) / shape[1] ** 0.5
+        elif len(shape) == 2:
+            t = torch.randn(shape, generator=g) / shape[1] ** 0.5
+        elif leaf == "correction":
+            t = 0.2 * torch.randn(shape, generator=g)
+        elif leaf == "sink":
+            t = 1.5 * torch.randn(shape, generator=g)
+        elif name.endswith(".f.b"):
+            t = 2.0 + 1.5 * torch.randn(shape, generator=g)
+        elif leaf == "b":
+            t = 0.4 * torch.randn(shape, generator=g)
+        else:                                                # norm weights
+            t = 1.0 + 0.2 * torch.randn(shape, generator=g)
+        out[name] = t.to(torch.bfloat16).float()
+    return out
