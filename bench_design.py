@@ -1,8 +1,9 @@
-"""``bench.py --design gufotar | pesivik | tisosun | gofezen``: prefill and decode throughput of a layer-list design at a few sizes that resemble
+"""``bench.py --design gufotar | pesivik | tisosun | gofezen | torutar``: prefill and decode throughput of a layer-list design at a few sizes that resemble
 a real model's layers (random weights, synthetic ids), beside the closest existing model of the framework (the
 uniform rotary decoder: same width, layer count, attention geometry and feed-forward width; for Tisosun the Gufotar
 layer-list model, the other design with recurrent layers beside attention layers; for Gofezen the Tisosun model, the
-other design of parallel blocks), plus every kernel of the
+other design of parallel blocks; for Torutar the Gofezen model, the other design of window attention, memories and gated
+routed experts), plus every kernel of the
 new path timed alone against its like kernel with the fraction of the measured roofline each reaches.
 
 Timing: CUDA events on the launching stream, >= 3 warm-up runs, a 256 MiB write between timed runs (larger than the
@@ -830,14 +831,19 @@ def gofezen_step_throughput(sz, batch, prompt, dev, dtype, flush) -> dict:
     """tokens/s of a whole-prompt step and of a decode step: Gofezen beside the Tisosun model (the other design of
     parallel blocks with recurrent layers and attention side by side with linear attention) of the same width, depth,
     attention geometry and dense feed-forward width."""
+    return _layered_steps((("gofezen", lambda m: build_gofezen(sz, batch, m, dev, dtype)),
+                           ("tisosun", lambda m: build_tisosun(sz, batch, m, dev, dtype))), sz, batch, prompt, flush)
+
+
+def _layered_steps(builders, sz, batch, prompt, flush) -> dict:
+    """Prefill and decode steps of layer-list models: ``builders`` = (name, max positions -> runner) pairs."""
     max_pos = prompt + 64
     out = {}
     gen = torch.Generator().manual_seed(0)
     ids = torch.randint(0, sz["vocab"], (batch, prompt), generator=gen)
     tok = [[int(t)] for t in torch.randint(0, sz["vocab"], (batch,), generator=gen)]
-    for name, build in (("gofezen", lambda: build_gofezen(sz, batch, max_pos, dev, dtype)),
-                        ("tisosun", lambda: build_tisosun(sz, batch, max_pos, dev, dtype))):
-        r = build()
+    for name, build in builders:
+        r = build(max_pos)
         r.enable_ragged_decode_graphs(widths=(batch,), ctx_buckets=(max_pos,))
         reqs = []
 
@@ -1062,6 +1068,244 @@ def gofezen_kernel_table(sz, batch, prompt, dev, dtype, flush, hbm_gbs, tflops) 
     return rows
 
 
+# ------------------------------------------------------------------------------------------------------ Torutar #
+U_SIZES = {
+    # attention layers: heads x head_dim on kv_heads, window + kept first tokens (every third of them reads the previous
+    # one's cache); a latent layer; matrix memories m_heads x (m_dim x m_vdim); routed experts + a shared one in every layer;
+    # the other columns are the Gofezen geometry of equal width, depth, attention shape, experts and memories
+    "small": dict(width=1024, layers=4, heads=16, kv_heads=4, head_dim=64, window=256, keep=4, q_rank=256, kv_rank=96, rot=32,
+                  l_dim=64, m_heads=16, m_dim=64, m_vdim=64, streams=4, taps=4, experts=16, top=2, e_ff=512, shared=1024,
+                  vocab=32000, r_heads=16, r_qk=4, r_dim=64, r_vdim=64, f_heads=16, f_dim=64, f_vdim=64, ff=2048),
+    "1b": dict(width=2048, layers=8, heads=16, kv_heads=4, head_dim=128, window=256, keep=4, q_rank=512, kv_rank=96, rot=32,
+               l_dim=128, m_heads=16, m_dim=128, m_vdim=128, streams=4, taps=4, experts=32, top=4, e_ff=512, shared=2048,
+               vocab=32000, r_heads=16, r_qk=4, r_dim=128, r_vdim=128, f_heads=16, f_dim=128, f_vdim=128, ff=4096),
+    "8b": dict(width=4096, layers=8, heads=32, kv_heads=8, head_dim=128, window=256, keep=4, q_rank=1024, kv_rank=96, rot=32,
+               l_dim=128, m_heads=32, m_dim=128, m_vdim=128, streams=4, taps=4, experts=64, top=4, e_ff=1024, shared=3072,
+               vocab=32000, r_heads=32, r_qk=8, r_dim=128, r_vdim=128, f_heads=32, f_dim=128, f_vdim=128, ff=7168),
+}
+
+
+def torutar_config(sz: dict) -> dict:
+    """Layers in the order attention, matrix memory, attention on the previous attention layer's cache, latent, ..."""
+    mlp = {"kind": "moe", "expert": {"ff": sz["e_ff"], "limit": 7.0}, "shared": {"ff": sz["shared"], "limit": 6.0},
+           "router": {"experts": sz["experts"], "top": sz["top"], "scale": 1.5}}
+    att = {"heads": sz["heads"], "kv_heads": sz["kv_heads"], "dim": sz["head_dim"], "vdim": sz["head_dim"],
+           "scale": 1.0 / math.sqrt(sz["head_dim"]), "mask": {"size": sz["window"], "keep_first": sz["keep"]},
+           "rot": {"dims": sz["head_dim"] // 2, "base": 10000.0}}
+    lat = {"heads": sz["heads"], "dim": sz["l_dim"], "rot_dim": sz["rot"], "vdim": sz["l_dim"], "q_rank": sz["q_rank"],
+           "kv_rank": sz["kv_rank"], "scale": 1.0 / math.sqrt(sz["l_dim"] + sz["rot"]), "rot": {"dims": sz["rot"], "base": 10000.0}}
+    mem = {"heads": sz["m_heads"], "dim": sz["m_dim"], "vdim": sz["m_vdim"], "gate_cap": 15.0}
+    order = [("attention", att), ("mlstm", mem), ("attention", None), ("latent_attention", lat)]
+    layers = []
+    for i in range(sz["layers"]):
+        kind, m = order[i % 4]
+        layers.append({"type": kind, "mixer": dict(att, kv_from=i - 2) if m is None else m, "mlp": mlp})
+    return {"architecture": "Torutar", "width": sz["width"], "vocab": sz["vocab"], "norm": {"eps": 1e-6}, "streams": sz["streams"],
+            "canon": {"taps": sz["taps"]}, "logit_scale": 0.5, "layers": layers}
+
+
+def build_torutar(sz, batch, max_positions, dev, dtype):
+    from lite_llama_b200.executor import ModelRunner
+    from lite_llama_b200.executor.layered_decoder import map_torutar_weights, parse_torutar_config, random_torutar_tensors
+
+    conf = parse_torutar_config(torutar_config(sz))
+    conf.validate()
+    weights = map_torutar_weights(conf, random_torutar_tensors(conf, seed=0), dev, dtype)
+    return ModelRunner(conf, weights, batch * max_positions, device=dev, dtype=dtype, max_requests=batch)
+
+
+def torutar_step_throughput(sz, batch, prompt, dev, dtype, flush) -> dict:
+    """tokens/s of a whole-prompt step and of a decode step: Torutar beside the Gofezen model (the other design of window
+    attention, linear-attention memories and gated routed experts) of the same width, depth, attention geometry, memory
+    sizes, expert count and expert width."""
+    return _layered_steps((("torutar", lambda m: build_torutar(sz, batch, m, dev, dtype)),
+                           ("gofezen", lambda m: build_gofezen(sz, batch, m, dev, dtype))), sz, batch, prompt, flush)
+
+
+def torutar_kernel_table(sz, batch, prompt, dev, dtype, flush, hbm_gbs, tflops) -> list[dict]:
+    """Every kernel of the Torutar path alone at the size's shapes beside its like kernel of the Gofezen path (latent
+    attention: of the Pesivik path), with the fraction of the measured roofline each reaches."""
+    import lite_llama_b200.kernels as K
+    from lite_llama_b200.executor.layered_decoder import split_plan
+    from lite_llama_b200.executor.ragged_batch import RaggedBatch
+
+    es = 2
+    W, H, G, D, win, keep = sz["width"], sz["heads"], sz["kv_heads"], sz["head_dim"], sz["window"], sz["keep"]
+    S, taps, E, top, eff, sff = sz["streams"], sz["taps"], sz["experts"], sz["top"], sz["e_ff"], sz["shared"]
+    T, ctx = batch * prompt, prompt
+    rows: list[dict] = []
+
+    def i32(v):
+        return torch.tensor(list(v), dtype=torch.int32, device=dev)
+
+    def rnd(*shape, dt=dtype, s=1.0):
+        return (torch.randn(*shape, device=dev) * s).to(dt)
+
+    def add(name, like, fn, nbytes=0, flops=0, like_fn=None, like_bytes=None, like_flops=None):
+        ms = timed(fn, flush)
+        row = {"kernel": name, "us": ms * 1e3}
+        if flops:
+            row.update(tflops=flops / ms / 1e9, frac=flops / ms / 1e9 / tflops, bound="tensor")
+        else:
+            row.update(gbs=nbytes / ms / 1e6, frac=nbytes / ms / 1e6 / hbm_gbs, bound="hbm")
+        if like_fn is not None:
+            lms = timed(like_fn, flush)
+            lf = like_flops if like_flops is not None else flops
+            lb = like_bytes if like_bytes is not None else nbytes
+            lfrac = lf / lms / 1e9 / tflops if flops else lb / lms / 1e6 / hbm_gbs
+            row.update(like=like, like_us=lms * 1e3, like_frac=lfrac,
+                       distance_ratio=(lfrac / row["frac"]) if row["frac"] else None)
+        rows.append(row)
+
+    p_start, p_ctx, p_slot = i32(range(0, T + 1, prompt)), i32([0] * batch), i32(range(batch))
+    d_start, d_ctx = i32(range(batch + 1)), i32([ctx] * batch)
+    pb = RaggedBatch.build([prompt] * batch, [0] * batch, range(batch), i32(range(T)), dev)
+    db = RaggedBatch.build([1] * batch, [ctx] * batch, range(batch), i32(range(batch)), dev)
+    # ---------------- streams: the write of one sublayer and the read of the next
+    for name, n in (("prompts", T), ("decode", batch)):
+        xs = torch.randn(n, S, W, device=dev)
+        y, z, zb, nw = rnd(n, W), rnd(n, W), rnd(W), rnd(W, s=0.1) + 1
+        ye, y2 = rnd(n, top, W), rnd(n, W)
+        rin, coef = torch.rand(S, device=dev), torch.rand(S + S * S, device=dev) * 0.3
+        resid = torch.randn(n, W, device=dev)
+        cw, tail = rnd(W, taps, s=0.3), torch.zeros(batch, taps - 1, W, dtype=dtype, device=dev)
+        conv = (cw, tail, d_ctx, p_slot) if name == "decode" else None
+        conv_bytes = W * taps * es + n * W * es * (2 * taps - 1) if conv else 0
+        like = lambda: K.branch_sum_residual(resid, y, None, z, None, y2, 1e-6, 0.6, want_act=False, scale_b=0.9, next_weight=nw)
+        lb = n * W * (8 + 3 * es + es)
+        add(f"stream_mix after a mixer ({name}; gate, {S} streams{', input convolution' if conv else ''})",
+            "branch_sum_residual (two scaled branches + feed-forward + next norm)",
+            lambda: K.stream_mix(xs, y, coef, rin, nw, 1e-6, gate=z, gate_bias=zb, conv=conv),
+            nbytes=n * W * (8 * S + 3 * es) + conv_bytes, like_fn=like, like_bytes=lb)
+        add(f"stream_mix after experts ({name}; {top} expert terms + shared, gate)",
+            "branch_sum_residual (two scaled branches + feed-forward + next norm)",
+            lambda: K.stream_mix(xs, ye, coef, rin, nw, 1e-6, addend=y2, gate=z, gate_bias=zb, conv=conv),
+            nbytes=n * W * (8 * S + (3 + top + 1) * es - es) + conv_bytes, like_fn=like, like_bytes=lb)
+    h = rnd(T, W)
+    cw, tail = rnd(W, taps, s=0.3), torch.zeros(batch, taps - 1, W, dtype=dtype, device=dev)
+    ch = 2 * sz["r_qk"] * sz["r_dim"] + sz["r_heads"] * sz["r_vdim"]
+    gproj, gcw, gtail = rnd(T, ch), rnd(ch, 4, s=0.5), torch.zeros(batch, 3, ch, dtype=dtype, device=dev)
+    gb = torch.zeros(ch, dtype=dtype, device=dev)
+    add("input convolution (prompts)", "causal convolution + SiLU of q', k', v'",
+        lambda: K.causal_conv_silu(h, 0, W, cw, None, tail, p_start, p_ctx, p_slot, activation=False, residual=True),
+        nbytes=T * W * 2 * es, like_fn=lambda: K.causal_conv_silu(gproj, 0, ch, gcw, gb, gtail, p_start, p_ctx, p_slot),
+        like_bytes=T * ch * 2 * es)
+    # ---------------- window attention with kept first tokens, sinks, gates
+    cols = -(-(H + 2 * G) * D // 8) * 8 + -(-H // 8) * 8
+    proj = rnd(T, cols, s=0.5)
+    kvw = 2 * G * D
+    pool = rnd(batch * (ctx + 1), kvw, s=0.5)
+    tab = torch.arange(batch * (ctx + 1), dtype=torch.int32, device=dev).view(batch, ctx + 1)
+    rows_p = tab[:, :ctx].reshape(-1).contiguous()
+    pos_p = i32(list(range(prompt)) * batch)
+    qn, kn, ones = rnd(D, s=0.1) + 1, rnd(D, s=0.1) + 1, torch.ones(D, dtype=dtype, device=dev)
+    rot = D // 2
+    cs = K.rope_table(pos_p, rot, 10000.0)
+    prep = T * ((2 * H + 2 * G) * D * es + 2 * G * D * es)
+    add("head_norm_rope_prepare (weights, halves rotation, value norm, cache write)", "head_norm_rope_prepare (unit-RMS of q and k)",
+        lambda: K.head_norm_rope_prepare(proj, pool, rows_p, cs, qn, kn, H, G, D, D, rot, 1e-6, "halves", True),
+        nbytes=prep + T * rot * 4, like_fn=lambda: K.head_norm_rope_prepare(proj, pool, rows_p, None, ones, ones, H, G, D, D, 0, 1e-6),
+        like_bytes=prep)
+    out = torch.empty(T, H * D, dtype=dtype, device=dev)
+    sink, gate = rnd(H), proj[:, -8 * (-(-H // 8)):][:, :H]
+    scale = 1.0 / math.sqrt(D)
+    seen = sum(min(t + 1, win + keep) for t in range(prompt))
+    lseen = sum(min(t + 1, win) for t in range(prompt))
+    add(f"window attention (prompts, window {win} + {keep} kept, sink, gate)", f"window attention (prompts, window {win})",
+        lambda: K.sink_attention(out, proj, pool, tab, p_start, p_ctx, p_slot, None, batch, prompt, sink, H, G, D, D, scale, 0.0,
+                                 window=win, keep_first=keep, gate=gate),
+        flops=4 * batch * H * D * seen,
+        like_fn=lambda: K.sink_attention(out, proj, pool, tab, p_start, p_ctx, p_slot, None, batch, prompt, None, H, G, D, D,
+                                         scale, 0.0, window=win), like_flops=4 * batch * H * D * lseen)
+    keys, lkeys = min(ctx + 1, win + keep), min(ctx + 1, win)
+    sp, per = split_plan(keys)
+    talk = rnd(H, H, s=0.2)
+    add(f"window attention (decode, {keys} of {ctx + 1} keys, sink, gate)", f"window attention, mixed heads (decode, {lkeys} keys)",
+        lambda: K.sink_attention(out, proj, pool, tab, d_start, d_ctx, p_slot, None, batch, 1, sink, H, G, D, D, scale, 0.0,
+                                 num_splits=sp, split_keys=per, window=win, keep_first=keep, gate=gate),
+        nbytes=batch * keys * kvw * es,
+        like_fn=lambda: K.mixed_head_attention(out, proj, pool, tab, d_start, d_ctx, p_slot, None, batch, talk, H, G, D, D, scale,
+                                               0.0, lkeys, window=win), like_bytes=batch * lkeys * kvw * es)
+    # ---------------- latent attention beside the Pesivik path's kernels (halves pairing, one gate per head)
+    qr, kr, lr, ld = sz["q_rank"], sz["kv_rank"], sz["rot"], sz["l_dim"]
+    LD = kr + lr
+    lproj = rnd(T, -(-(qr + kr + lr + H * ld) // 8) * 8, s=0.5)
+    lpool = rnd(batch * (ctx + 1), LD, s=0.5)
+    wq, wkv = rnd(qr, s=0.1) + 1, rnd(kr, s=0.1) + 1
+    lcs = K.rope_table(pos_p, lr, 10000.0)
+    add("latent_prepare (neighbour pairs)", "latent_prepare (halves)",
+        lambda: K.latent_prepare(lproj, lpool, rows_p, lcs, wq, wkv, qr, kr, lr, lr, 1e-6, "neighbours"),
+        nbytes=T * ((2 * qr + kr + lr) * es + LD * es),
+        like_fn=lambda: K.latent_prepare(lproj, lpool, rows_p, lcs, wq, wkv, qr, kr, lr, lr, 1e-6))
+    q, qa = rnd(T, H * (ld + lr), s=0.5), torch.empty(T, H * LD, dtype=dtype, device=dev)
+    add("rope_heads (neighbour pairs)", "rope_heads (halves)",
+        lambda: K.rope_heads(qa[:, kr:], LD, q[:, ld:], ld + lr, lcs, H, lr, lr, "neighbours"), nbytes=T * H * lr * 2 * es,
+        like_fn=lambda: K.rope_heads(qa[:, kr:], LD, q[:, ld:], ld + lr, lcs, H, lr, lr))
+    lat, o, uv = rnd(T, H * kr, s=0.5), torch.empty(T, H * ld, dtype=dtype, device=dev), rnd(H, ld, kr, s=0.1)
+    lgate = lproj[:, qr + kr + lr:]
+    add("head_linear (values out of the latent, element gate)", "head_linear (head gate)",
+        lambda: K.head_linear(o, ld, lat, kr, uv, lgate, True), flops=2 * T * H * ld * kr,
+        like_fn=lambda: K.head_linear(o, ld, lat, kr, uv, lgate))
+    # ---------------- matrix memory beside the delta rule and the chunked fixed-decay memory
+    MH, MD, MV = sz["m_heads"], sz["m_dim"], sz["m_vdim"]
+    n_in = MH * (2 * MD + 2 * MV) + 2 * MH
+    mproj = rnd(T, -(-n_in // 8) * 8, s=0.5)
+    mst = torch.zeros(batch, MH, K.mlstm_head_floats(MD, MV), device=dev)
+    bi, bf = rnd(MH), rnd(MH) + 3
+    mq, mk, mv = mproj[:, :MH * MD], mproj[:, MH * MD:2 * MH * MD], mproj[:, 2 * MH * MD:2 * MH * MD + MH * MV]
+    mi, mf = mproj[:, n_in - 2 * MH:n_in - MH], mproj[:, n_in - MH:n_in]
+
+    def memory(n, b):
+        return K.mlstm(mst, mq[:n], mk[:n], mv[:n], mi[:n], mf[:n], bi, bf, b, MH, MD, MV, 15.0, MD ** -0.5)
+
+    RH, RQ, RD, RV = sz["r_heads"], sz["r_qk"], sz["r_dim"], sz["r_vdim"]
+    dch = 2 * RQ * RD + RH * RV
+    dproj, dst = rnd(T, dch + 2 * RH, s=0.5), torch.zeros(batch, RH, RD, RV, device=dev)
+    dtb, alog = rnd(RH) - 1, rnd(RH, s=0.5) - 1
+
+    def delta(n, start, cx):
+        return K.gated_linear_scan("delta_rule", dst, dproj[:n, :RQ * RD], dproj[:n, RQ * RD:2 * RQ * RD], dproj[:n, 2 * RQ * RD:dch],
+                                   start, cx, p_slot, RH, RQ, RD, RV, c0=dtb, c1=alog, p0=dproj[:n, dch:dch + RH],
+                                   p1=dproj[:n, dch + RH:], q_scale=RD ** -0.5)
+
+    m_bytes = T * (n_in * es - MH * MV * es + MH * MV * 4) + batch * MH * MD * MV * 4
+    add("mlstm (prompts, 64-token chunks)", "gated_linear_scan, delta rule (prompts)", lambda: memory(T, pb), nbytes=m_bytes,
+        like_fn=lambda: delta(T, p_start, p_ctx), like_bytes=T * ((dch + 2 * RH) * es + RH * RV * 4) + batch * RH * RD * RV * 4)
+    tx = rnd(T, RH * (2 * RD + RV), s=0.5)
+    dec = torch.tensor([1.0 - 2.0 ** (-2 - 6 * i / RH) for i in range(RH)], dtype=torch.float32, device=dev)
+    lms = timed(lambda: K.decay_attention(tx, dst, dec, p_start, p_ctx, p_slot, RH, RD, RV, prompt), flush)
+    lfrac = (T * (RH * (2 * RD + RV) * es + RH * RV * 4) + batch * RH * RD * RV * 4) / lms / 1e6 / hbm_gbs
+    rows.append(dict(rows[-1], like="decay_attention (prompts, 64-token chunks)", like_us=lms * 1e3, like_frac=lfrac,
+                     distance_ratio=lfrac / rows[-1]["frac"]))
+    add("mlstm (decode)", "gated_linear_scan, delta rule (decode)", lambda: memory(batch, db), nbytes=batch * MH * (MD * MV + MD) * 8,
+        like_fn=lambda: delta(batch, d_start, d_ctx), like_bytes=batch * RH * RD * RV * 8)
+    yf, nw1, nw2 = torch.randn(T, MH * MV, device=dev), rnd(MH * MV, s=0.1) + 1, rnd(MV, s=0.1) + 1
+    mgate = mproj[:, MH * 2 * MD + MH * MV:MH * 2 * MD + 2 * MH * MV]
+    add("head_norm_gate (weight per head, sigmoid gate)", "head_norm_gate (shared weight, SiLU gate)",
+        lambda: K.head_norm_gate(yf, nw1, MH, 1e-6, mgate, "sigmoid"), nbytes=T * MH * MV * (4 + 2 * es),
+        like_fn=lambda: K.head_norm_gate(yf, nw2, MH, 1e-6, mgate))
+    # ---------------- experts
+    gu = rnd(T, 2 * sff)
+    add("swiglu_scaled (clamped unit)", "swiglu_scaled (SiLU)",
+        lambda: K.swiglu_scaled(gu[:, :sff], gu[:, sff:], form="clamped", limit=6.0), nbytes=T * sff * 3 * es,
+        like_fn=lambda: K.swiglu_scaled(gu[:, :sff], gu[:, sff:]))
+    x, router, corr = rnd(T, W, s=0.5), rnd(E, W, s=W ** -0.5), rnd(E, s=0.02)
+    add("route_sigmoid_groups (softmax scores, scaled)", "route_sigmoid_groups (sigmoid scores kept)",
+        lambda: K.route_sigmoid_groups(x, router, corr, top, scores="softmax", scale=1.5), flops=2 * T * E * W,
+        like_fn=lambda: K.route_sigmoid_groups(x, router, None, top, 1, 1, renormalize=False))
+    wts, ids = K.route_sigmoid_groups(x, router, corr, top, scores="softmax", scale=1.5)
+    wgu, wdn = rnd(E, 2 * eff, W, s=W ** -0.5), rnd(E, W, eff, s=eff ** -0.5)
+    for name, n in (("prompts", T), ("decode", batch)):
+        xn, wn, idn = x[:n], wts[:n].contiguous(), ids[:n].contiguous()
+        cost = dict(flops=2 * n * top * 3 * eff * W) if name == "prompts" else \
+            dict(nbytes=len(set(idn.flatten().tolist())) * 3 * eff * W * es)
+        add(f"grouped_experts, clamped unit in the epilogue, terms handed out ({name})",
+            f"grouped_experts, gated, weight on the input ({name})",
+            lambda: K.grouped_experts(xn, wgu, wdn, wn, idn, activation="clamped", gated=True, limit=7.0, reduce=False), **cost,
+            like_fn=lambda: K.grouped_experts(xn, wgu, wdn, wn, idn, activation="silu", gated=True, weight_on_input=True))
+    return rows
+
+
 def run(args) -> None:
     from bench import ClockSampler, peaks
 
@@ -1073,7 +1317,8 @@ def run(args) -> None:
     sizes = [s for s in (args.design_sizes or "small,1b,8b").split(",") if s]
     table, steps, kernels = {"pesivik": (P_SIZES, pesivik_step_throughput, pesivik_kernel_table),
                              "tisosun": (T_SIZES, tisosun_step_throughput, tisosun_kernel_table),
-                             "gofezen": (G_SIZES, gofezen_step_throughput, gofezen_kernel_table)}.get(
+                             "gofezen": (G_SIZES, gofezen_step_throughput, gofezen_kernel_table),
+                             "torutar": (U_SIZES, torutar_step_throughput, torutar_kernel_table)}.get(
         args.design, (SIZES, step_throughput, kernel_table))
     result = {"design": args.design, "dtype": "bf16", "data": "synthetic ids, random weights", "peaks": {"hbm_gbs": hbm_gbs, "bf16_tflops": tflops, "source": src},
               "batch": args.batch, "prompt_len": args.prompt_len, "l2_policy": "256 MiB written between timed runs", "sizes": {}}

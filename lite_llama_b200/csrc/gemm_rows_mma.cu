@@ -146,14 +146,29 @@ __global__ void __launch_bounds__(128) rows_gemm_mma_kernel(RowsArgs a) {
     }
     T* dst = (T*)crow[r];
     const T* ge = nullptr;                                     // the row's element gates of this head
-    if (!GROUPED && a.gate_elements) ge = (const T*)a.gate + ((int64_t)blockIdx.y * BM + r) * a.gs + blockIdx.z * a.n;
+    uint32_t gz[NT];                                           // their logits, two columns each: all loads in flight at once
+    if (!GROUPED && a.gate_elements) {
+      ge = (const T*)a.gate + ((int64_t)blockIdx.y * BM + r) * a.gs + blockIdx.z * a.n;
+#pragma unroll
+      for (int j = 0; j < NT; ++j) {
+        const int64_t col = n0 + wn * (NT * 8) + j * 8 + 2 * tq;
+        gz[j] = 0u;
+        T* e = reinterpret_cast<T*>(&gz[j]);
+        if (col + 1 < a.n && (((uintptr_t)(ge + col)) & 3) == 0) gz[j] = *reinterpret_cast<const uint32_t*>(ge + col);
+        else {
+          if (col < a.n) e[0] = ge[col];
+          if (col + 1 < a.n) e[1] = ge[col + 1];
+        }
+      }
+    }
 #pragma unroll
     for (int j = 0; j < NT; ++j) {
       const int64_t col = n0 + wn * (NT * 8) + j * 8 + 2 * tq;
       float v0 = acc[mi][j][half * 2], v1 = acc[mi][j][half * 2 + 1];
       if (!GROUPED && ge) {
-        if (col < a.n) v0 *= 1.0f / (1.0f + expf(-to_f32(ge[col])));
-        if (col + 1 < a.n) v1 *= 1.0f / (1.0f + expf(-to_f32(ge[col + 1])));
+        const T* e = reinterpret_cast<const T*>(&gz[j]);
+        v0 = __fdividef(v0, 1.0f + __expf(-to_f32(e[0])));
+        v1 = __fdividef(v1, 1.0f + __expf(-to_f32(e[1])));
       }
       if (GROUPED && a.act == 2) {
         if (col + 1 < a.n) dst[col >> 1] = from_f32<T>(a.unit(v0, v1) * g);

@@ -180,7 +180,9 @@ __global__ void __launch_bounds__(256) stream_kernel(StreamArgs a) {
       }
       for (int j = 0; j < keep - 1; ++j) {
         float v[C];
-        load_c<C>(tail + (int64_t)(j + 1) * n + i, v);
+#pragma unroll
+        for (int c = 0; c < C; ++c) v[c] = 0.f;
+        if (ctx - keep + j + 1 >= 0) load_c<C>(tail + (int64_t)(j + 1) * n + i, v);
         store_c<C>(tail + (int64_t)j * n + i, v);
       }
       if (keep > 0) store_c<C>(tail + (int64_t)(keep - 1) * n + i, h);
