@@ -60,7 +60,7 @@ __device__ __forceinline__ void store_c(T* p, const float (&v)[C]) {
 }
 
 template <typename T, int S, int C, bool EMBED>      // S = streams (8: up to eight, a.s of them)
-__global__ void __launch_bounds__(256) stream_kernel(StreamArgs a) {
+__global__ void __launch_bounds__(512) stream_kernel(StreamArgs a) {
   pdl_prologue();
   extern __shared__ __align__(16) float u_row[];     // [n]
   __shared__ float red[32];
@@ -194,7 +194,8 @@ __global__ void __launch_bounds__(256) stream_kernel(StreamArgs a) {
 template <typename T, int C, bool EMBED>
 int launch_stream(const StreamArgs& a, int64_t tokens, cudaStream_t st) {
   const int64_t per = cdiv64(a.n, C);
-  const int threads = per >= 256 ? 256 : (int)(cdiv64(per, 32) * 32);
+  const int64_t most = tokens <= 2 * b2l_num_sms() ? 512 : 256;        // few tokens: the latency of one row is all there is
+  const int threads = per >= most ? (int)most : (int)(cdiv64(per, 32) * 32);
   const size_t smem = (size_t)a.n * sizeof(float);
   B2L_REQUIRE((int64_t)smem <= b2l_max_smem_optin() - 1024, "stream kernels: rows of %lld elements", (long long)a.n);
 #define B2L_STREAM(S)                                                                                     \
