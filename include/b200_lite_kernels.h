@@ -319,8 +319,8 @@ int b2l_moe_gemm_mma(void* c, const void* a, const void* w, const void* slot_wei
  * weights. */
 int b2l_moe_route_sigmoid_groups(void* weights_f32, void* ids_i32, const void* x, int64_t x_row_stride,
                                  const void* router_w, const void* bias, const void* logits_f32, int64_t tokens,
-                                 int num_experts, int64_t k, int top_k, int groups, int keep, int renormalize,
-                                 int softmax, float scale, int dtype, void* stream);
+                                 int num_experts, int64_t k, int top_k, int groups, int keep, int group_best,
+                                 int renormalize, int softmax, float scale, int dtype, void* stream);
 /* y_f32[m, n] = x[m, k] . w[n, k]^T: 16-bit operands on the tensor cores, the fp32 sums stored unrounded (router
  * logits); operands as b2l_rows_gemm_mma_ok asks. */
 int b2l_linear_f32out_mma(void* y_f32, const void* x, const void* w, int64_t m, int64_t n, int64_t k,
@@ -329,7 +329,7 @@ int b2l_linear_f32out_mma(void* y_f32, const void* x, const void* w, int64_t m, 
  * fp64 (csrc/latent_attention.cu); one table per step serves every layer with these rotary constants. */
 int b2l_rope_table(void* cos_sin_f32, const void* pos_i32, int64_t tokens, int rot_dims, float rot_base, void* stream);
 /* Latent attention, per token of the fused down-projection row [a: q_rank | b: kv_rank | r: rot_dim | ...]:
- * a <- rmsnorm(a) * q_norm_weight in place; pool row kv_rows[t] = [rmsnorm(b) * kv_norm_weight | r with its first
+ * a <- rmsnorm(a) * q_norm_weight in place (q_rank 0: no query latent); pool row kv_rows[t] = [rmsnorm(b) * kv_norm_weight | r with its first
  * rot_dims entries rotated by the token's row of cos_sin_f32 (pairing 1: entry i pairs with i + rot_dims / 2, 0:
  * neighbours 2i, 2i + 1)]. */
 int b2l_latent_prepare(void* proj, int64_t proj_row_stride, void* pool, int64_t pool_row_stride,
@@ -376,12 +376,20 @@ int b2l_attn_prepare(void* qkv, int64_t qkv_row_stride, void* kv_pool, int64_t k
                      const void* pos_i32, const void* q_norm_weight, const void* k_norm_weight, const void* v_first_in,
                      void* v_first_out, const void* v_lambda, int64_t tokens, int q_cols, int k_cols, int v_cols,
                      float eps, float gain_coef, float gain_every, int dtype, void* stream);
+/* Keys that serve as values too, per token of [q: q_cols | k: k_cols | ...] (csrc/attention_sink.cu): q <- rmsnorm(q) *
+ * query_weight_f32 * gain(pos) in place (the weight holds the key norm's channel weights as well), pool row kv_rows[t] =
+ * [k as projected | at factor_col: 1 / rms(k) as fp32]. */
+int b2l_norm_query_keep_key(void* qk, int64_t qk_row_stride, void* kv_pool, int64_t kv_row_stride,
+                            const void* kv_rows_i32, const void* pos_i32, const void* query_weight_f32, int64_t tokens,
+                            int q_cols, int k_cols, int factor_col, float eps, float gain_coef, float gain_every,
+                            int dtype, void* stream);
 /* Soft-capped attention with an optional per-head sink over the pool (csrc/attention_sink.cu).  num_splits == 0: tiled
  * mode for sequences of up to max_q_len new tokens; num_splits > 0: every listed sequence brings one token, its keys
  * (from the first one it sees) are cut into num_splits ranges of split_keys and merged (workspace:
  * b2l_sink_attention_workspace_bytes).  window > 0: token p sees keys p - window + 1 .. p only, and with keep_first > 0
  * also the sequence's first keep_first positions; gate (nullable) [tokens, >= heads]: head h's output times
- * sigmoid(gate[t, h]); block > 0 (window <= 0):
+ * sigmoid(gate[t, h]) (gate_elements: a gate [tokens, heads * v_head_dim], element by element); key_factor_col >= 0:
+ * every pool row holds one fp32 number at that column which multiplies its keys' scores; block > 0 (window <= 0):
  * token p sees keys floor(p / block) * block .. p only.  v_col0 < 0: a pool
  * row is [keys | values]; v_col0 >= 0: the values start at that column (0: they are the keys' leading columns).
  * v_blocks > 1 (num_splits > 0 only): v_blocks neighbouring blocks of v_head_dim value columns in one call, each as
@@ -392,9 +400,9 @@ int b2l_sink_attention(void* out, int64_t out_row_stride, const void* q, int64_t
                        const void* seq_ctx, const void* seq_slot, const void* seq_list, int64_t num_seqs,
                        int max_q_len, const void* sink, int heads, int kv_heads, int head_dim, int v_head_dim,
                        float scale, float softcap, int window, int keep_first, int block, int v_col0,
-                       int v_head_stride, int v_blocks, const void* gate, int64_t gate_row_stride, int num_splits,
-                       int split_keys, void* workspace, int64_t workspace_bytes, int dtype,
-                       void* stream);
+                       int v_head_stride, int v_blocks, const void* gate, int64_t gate_row_stride, int gate_elements,
+                       int key_factor_col, int num_splits, int split_keys, void* workspace, int64_t workspace_bytes,
+                       int dtype, void* stream);
 /* One new token per listed sequence, the heads' softmax weights mixed across heads before the values:
  * p'_h(j) = sum_g mix[h, g] p_g(j), out_h = sum_j p'_h(j) v_kv(h)(j).  mix [heads, heads] has q's element type.  max_keys
  * bounds the keys any listed token sees (window, or context + 1); the workspace holds num_seqs * heads * max_keys fp32
@@ -464,10 +472,22 @@ int b2l_head_norm_gate(void* out, const void* y_f32, const void* gate, int64_t g
 int b2l_head_mix(void* out, const void* wide, int64_t wide_row_stride, const void* mix, int64_t rows, int heads,
                  int kv_heads, int per_call, int vdim, int dtype, void* stream);
 /* out[r, :] = silu(s_r * gate[r, :]) * (s_r * up[r, :]) * sigmoid(z[r]); in_scale_f32 [rows] and z (one value per row,
- * row stride given) are nullable.  form 1: the clamped unit g' sigmoid(alpha g') (u' + 1) instead of silu(g) u. */
+ * row stride given) are nullable.  form 1: the clamped unit g' sigmoid(alpha g') (u' + 1) instead of silu(g) u;
+ * form 2: gelu(g) u, tanh form. */
 int b2l_swiglu_scaled(void* out, int64_t out_row_stride, const void* gate, int64_t gate_row_stride, const void* up,
                       int64_t up_row_stride, const void* in_scale_f32, const void* z, int64_t z_row_stride, int64_t rows,
                       int64_t n, int form, float limit, float alpha, int dtype, void* stream);
+
+/* Residual of designs whose sublayers read an element-wise norm tanh(alpha x) * w + b and add their result as it is
+ * (csrc/tanh_norm_stream.cu).  Per element: v = residual_f32 (first 1: 0) + y (+ addend) (+ embed_scale * embed[token])
+ * (+ step); residual_f32 = v; act = tanh(alpha v) * w + b (nullable).  y [tokens, n] with top 0, else [tokens, top, n]: the
+ * weighted outputs of a token's chosen experts ids_i32 [tokens, top], where ids >= experts stand for their input:
+ * weights_f32 * x instead.  rows_i32 (nullable): only these tokens, act [num_rows, n], the residual is not written. */
+int b2l_tanh_norm_stream(void* residual_f32, void* act, const void* y, int64_t y_row_stride, int top,
+                         const void* ids_i32, const void* weights_f32, int experts, const void* x, int64_t x_row_stride,
+                         const void* addend, const void* tokens_i32, const void* embed, int64_t vocab,
+                         float embed_scale, const void* step, int first, const void* alpha, const void* w,
+                         const void* b, const void* rows_i32, int64_t num_rows, int64_t n, int dtype, void* stream);
 
 /* Matrix memory with exponential gates (csrc/mlstm.cu); state_f32 [slots, heads, b2l_mlstm_head_floats] = per head
  * [S: dim x vdim | n: dim | m | pad], advanced in place; y_f32 [tokens, heads * vdim].  With i = cap tanh((zi + bi) / cap),

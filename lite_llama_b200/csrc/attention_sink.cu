@@ -7,8 +7,15 @@
 // A sliding window (`window` > 0) limits token p to the keys p - window + 1 .. p; a block-diagonal mask (`block` > 0)
 // to the keys of its own run of `block` positions, floor(p / block) * block .. p (runs are counted from position 0).
 // `keep` > 0 (with a window): the sequence's first `keep` positions stay visible to every later token.  `gate`
-// (nullable, [tokens, >= heads]): head h's output is multiplied by sigmoid(gate[t, h]).
+// (nullable, [tokens, >= heads]): head h's output is multiplied by sigmoid(gate[t, h]), or, with `gate_elements`, element
+// d of head h by sigmoid(gate[t, h * Dv + d]).
+// `key_factor_col` >= 0: every pool row carries one fp32 number at that column (in elements of T) that multiplies the
+// scores of its keys.  A key norm without per-head statistics is such a number (the channel weights go into the query),
+// so a row can hold the keys as projected once and serve as keys and values (`v_col0` = 0, `v_hstride` = D).
+// Whenever the values are leading columns of the keys, the kernels stage one tile and read it twice.
 //
+//   norm_query_keep_key   per token: whole-row RMS norm of q with both norms' channel weights and the query gain, the
+//                  keys as projected plus their norm's statistic into the cache row
 //   attn_prepare   per token: whole-row RMS norm of q and of k (one statistic over ALL heads, plain weight),
 //                  position-dependent query gain, value mixing with an earlier layer's values, K|V cache write
 //   sink_attention sequence s brings q_len new tokens after ctx cached ones; token i sees cache positions 0..ctx+i
@@ -51,8 +58,17 @@ struct AttnArgs {
                                // one kv head (not tokens), blockIdx.x is a key range, results go to `part`
   float scale, softcap;
   int keep;                    // window only: key positions below `keep` are visible to every later token
-  const void* gate; int64_t gate_stride;      // per-head logistic output gate (nullable)
+  const void* gate; int64_t gate_stride;      // logistic output gate, per head or per element (nullable)
+  int gate_elements;
+  int key_factor_col;          // < 0: none; else the column of a pool row's fp32 score factor
+  int shared;                  // the values of a kv head are the leading Dv columns of its keys
 };
+
+// fp32 score factor of pool row `row`
+template <typename T>
+__device__ __forceinline__ float key_factor(const AttnArgs& a, int64_t row) {
+  return *reinterpret_cast<const float*>((const T*)a.kv + row * a.kv_stride + a.key_factor_col);
+}
 
 // first key position the token at `pos` sees (may be negative under a window: callers clamp where they index);
 // non-decreasing in pos for every mask kind, which the tile-level bounds below rely on
@@ -82,7 +98,9 @@ __global__ void __launch_bounds__(kWarps * 32) sink_attention_kernel(AttnArgs a)
   const int D = a.D, Dv = a.Dv, per = a.H / a.G;
   float* qs = smem;                              // [kRows][D]
   float* ks = qs + kRows * D;                    // [kKeys][D + 1]
-  float* vs = ks + kKeys * (D + 1);              // [kKeys][Dv]
+  float* kf = ks + kKeys * (D + 1);              // [kKeys] score factors
+  float* vs = a.shared ? ks : kf + kKeys;        // [kKeys][Dv], or the keys' own tile
+  const int vp = a.shared ? D + 1 : Dv;          // its pitch
   const int z = blockIdx.z, s = a.seq_list ? a.seq_list[z] : z;
   const int start = a.seq_start[s], qlen = a.seq_start[s + 1] - start, ctx = a.seq_ctx[s];
   const int64_t slot = a.seq_slot[s];
@@ -126,7 +144,11 @@ __global__ void __launch_bounds__(kWarps * 32) sink_attention_kernel(AttnArgs a)
       const bool in = j < nk && (k0 + j >= key_lo || k0 + j < keep_hi);       // positions no row sees may have no row
       ks[j * (D + 1) + d] = in ? to_f32(kv[(int64_t)trow[k0 + j] * a.kv_stride + g * D + d]) : 0.f;
     }
-    for (int i = tid; i < kKeys * Dv; i += blockDim.x) {
+    if (a.key_factor_col >= 0 && tid < kKeys) {
+      const bool in = tid < nk && (k0 + tid >= key_lo || k0 + tid < keep_hi);
+      kf[tid] = in ? key_factor<T>(a, trow[k0 + tid]) : 0.f;
+    }
+    for (int i = a.shared ? kKeys * Dv : tid; i < kKeys * Dv; i += blockDim.x) {
       const int j = i / Dv, d = i - j * Dv;
       const bool in = j < nk && (k0 + j >= key_lo || k0 + j < keep_hi);
       vs[i] = in ? to_f32(kv[(int64_t)trow[k0 + j] * a.kv_stride + a.v_col0 + g * a.v_hstride + d]) : 0.f;
@@ -148,6 +170,7 @@ __global__ void __launch_bounds__(kWarps * 32) sink_attention_kernel(AttnArgs a)
       const int row_lo = first_visible(a, row_pos[i]);
       if (row_lo >= k0 + nk && k0 >= keep_hi) continue;      // warp-uniform: the row's window starts after this tile
       float sv = sc[i] * a.scale;
+      if (a.key_factor_col >= 0) sv *= kf[lane];
       if (a.softcap > 0.f) sv = a.softcap * tanhf(sv * inv_cap);
       const bool ok = lane < nk && k0 + lane <= row_pos[i] && (k0 + lane >= row_lo || k0 + lane < keep_hi);
       sv = ok ? sv : -INFINITY;
@@ -165,7 +188,7 @@ __global__ void __launch_bounds__(kWarps * 32) sink_attention_kernel(AttnArgs a)
 #pragma unroll
         for (int j = 0; j < DVJ; ++j) {
           const int d = lane + 32 * j;
-          if (d < Dv) acc[i][j] = fmaf(pk, vs[kk * Dv + d], acc[i][j]);
+          if (d < Dv) acc[i][j] = fmaf(pk, vs[kk * vp + d], acc[i][j]);
         }
       }
     }
@@ -183,12 +206,17 @@ __global__ void __launch_bounds__(kWarps * 32) sink_attention_kernel(AttnArgs a)
         den = l[i] * num + expf(sk - mf);
       }
       float inv = num / den;
-      if (a.gate) inv *= gate_of(to_f32(((const T*)a.gate)[(int64_t)(start + t0 + tl) * a.gate_stride + h]));
+      const T* gr = a.gate ? (const T*)a.gate + (int64_t)(start + t0 + tl) * a.gate_stride : nullptr;
+      if (gr && !a.gate_elements) inv *= gate_of(to_f32(gr[h]));
       T* o = (T*)a.out + (int64_t)(start + t0 + tl) * a.out_stride + h * Dv;
 #pragma unroll
       for (int j = 0; j < DVJ; ++j) {
         const int d = lane + 32 * j;
-        if (d < Dv) o[d] = from_f32<T>(acc[i][j] * inv);
+        if (d < Dv) {
+          float v = acc[i][j] * inv;
+          if (a.gate_elements) v *= gate_of(to_f32(gr[h * Dv + d]));
+          o[d] = from_f32<T>(v);
+        }
       }
     }
   }
@@ -202,6 +230,9 @@ __global__ void __launch_bounds__(kWarps * 32) sink_attention_kernel(AttnArgs a)
 // O += P V run on mma.sync m16n8k16 with fp32 accumulators, the soft cap is applied to the fp32 scores, the online
 // softmax works in the log2 domain, the sink joins the denominator once at the end.  Keys 0 .. ctx + t (cached prefix
 // + the portion itself) are visible to token t.  Needs D, Dv multiples of 8 and <= 128, 16-byte aligned pool rows.
+// When the values are the keys' leading columns (SHARED) there is one tile per stage and O += P V reads it transposed.
+// Head sizes up to 320 / 256 run in this form (latent rows); with more than 128 value columns the tile is 32 keys and Q
+// stays in shared memory, which leaves the registers to the output accumulator.
 constexpr int kTileM = 64, kTileN = 64;
 constexpr float kLog2e = 1.4426950408889634f;
 
@@ -216,15 +247,32 @@ __device__ __forceinline__ float tanh_fast(float x) {
 __device__ __forceinline__ void cp_async_16(uint32_t saddr, const void* g) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(saddr), "l"(g) : "memory");
 }
+__device__ __forceinline__ void cp_async_4(uint32_t saddr, const void* g) {
+  asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(saddr), "l"(g) : "memory");
+}
 __device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
 template <int N> __device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
 
-template <typename T, int DP, int DVP>
+template <int DP, int DVP, bool SHARED>
+struct MmaTile {
+  static constexpr bool kQShared = DVP > 128;                    // Q fragments are re-read from shared memory
+  static constexpr int N = kQShared ? 32 : kTileN;               // keys per tile
+  static constexpr int KP = (DP + 8) * 2, VP = SHARED ? KP : (DVP + 8) * 2;      // row pitches in bytes
+  static constexpr int kStage = N * (KP + (SHARED ? 0 : VP));    // one K tile + one V tile (or the one both use)
+  static constexpr int kFactors = 2 * kStage;                    // two stages, then [2][N] score factors, then Q
+  static constexpr int kQ = kFactors + 2 * N * 4;
+  static constexpr int kBytes = kQ + (kQShared ? kTileM * KP : 0);
+};
+
+template <typename T, int DP, int DVP, bool SHARED>
 __global__ void __launch_bounds__(128) sink_attention_mma_kernel(AttnArgs a) {
   pdl_prologue();
   extern __shared__ __align__(16) uint8_t smem_raw[];
-  constexpr int KP = (DP + 8) * 2, VP = (DVP + 8) * 2;          // row pitches in bytes
-  constexpr int kStage = kTileN * (KP + VP);                    // one K tile + one V tile; two stages
+  using Tile = MmaTile<DP, DVP, SHARED>;
+  constexpr int KP = Tile::KP, VP = Tile::VP, kStage = Tile::kStage, kTileN = Tile::N;
+  constexpr bool QS = Tile::kQShared;
+  float* factors = reinterpret_cast<float*>(smem_raw + Tile::kFactors);
+  const bool has_factor = a.key_factor_col >= 0;
   const int D = a.D, Dv = a.Dv, per = a.H / a.G;
   const int z = blockIdx.z, s = a.seq_list ? a.seq_list[z] : z;
   const int start = a.seq_start[s], qlen = a.seq_start[s + 1] - start, ctx = a.seq_ctx[s];
@@ -263,8 +311,18 @@ __global__ void __launch_bounds__(128) sink_attention_mma_kernel(AttnArgs a) {
   auto row_of = [&](int k) { return (k < key_hi && (k >= tile_lo || k < keep_hi)) ? (hr ? axis.key(k) : k) : -1; };
   const T* q = (const T*)a.q;
   const T* kv = (const T*)a.kv;
-  uint32_t qf[DP / 16][4];
-  {
+  uint32_t qf[QS ? 1 : DP / 16][4];
+  if constexpr (QS) {                                            // rows past the end and columns past D are zero
+    constexpr int C2 = DP / 2;                                   // 4-byte column pairs
+    for (int i = tid; i < kTileM * C2; i += 128) {
+      const int r = i / C2, c = (i - r * C2) * 2;
+      uint32_t v = 0u;
+      if (r < t_count && c < D)
+        v = *reinterpret_cast<const uint32_t*>(hr ? q + (int64_t)start * a.q_stride + (h_base + r) * D + c
+                                                  : q + (int64_t)(start + t0 + r) * a.q_stride + h * D + c);
+      *reinterpret_cast<uint32_t*>(smem_raw + Tile::kQ + r * KP + c * 2) = v;
+    }
+  } else {
     const T* q0 = hr ? q + (int64_t)start * a.q_stride + (h_base + (ok0 ? r0 : 0)) * D
                      : q + (int64_t)(start + t0 + (ok0 ? r0 : 0)) * a.q_stride + h * D;
     const T* q1 = hr ? q + (int64_t)start * a.q_stride + (h_base + (ok1 ? r1 : 0)) * D
@@ -292,8 +350,9 @@ __global__ void __launch_bounds__(128) sink_attention_mma_kernel(AttnArgs a) {
     uint8_t* kdst = smem_raw + st * kStage;
     uint8_t* vdst = kdst + kTileN * KP;
     // the pool rows of this thread's copies first (independent loads), then the copies
-    constexpr int JK = kTileN * (DP / 8) / 128, JV = kTileN * (DVP / 8) / 128;
-    int rk[JK], rv[JV];
+    constexpr int JK = kTileN * (DP / 8) / 128, JV = SHARED ? 0 : kTileN * (DVP / 8) / 128;
+    static_assert(kTileN * (DP / 8) % 128 == 0, "whole copies per thread");
+    int rk[JK], rv[JV + 1];
 #pragma unroll
     for (int j = 0; j < JK; ++j) {
       const int r = (tid + 128 * j) / (DP / 8);
@@ -322,6 +381,12 @@ __global__ void __launch_bounds__(128) sink_attention_mma_kernel(AttnArgs a) {
       else
         *reinterpret_cast<uint4*>(vdst + r * VP + c * 2) = make_uint4(0u, 0u, 0u, 0u);
     }
+    if (has_factor && tid < kTileN) {
+      const int k = row_of(k0 + tid);
+      float* dst = factors + st * kTileN + tid;
+      if (k >= 0) cp_async_4(smem_u32(dst), kv + (int64_t)trow[k] * a.kv_stride + a.key_factor_col);
+      else *dst = 0.f;
+    }
     cp_async_commit();
   };
   const int k_start = (keep_hi > 0 && k_first > 0) ? 0 : k_first;
@@ -332,7 +397,7 @@ __global__ void __launch_bounds__(128) sink_attention_mma_kernel(AttnArgs a) {
     if (more) issue(kn, (it + 1) & 1);                           // the next tile flies while this one is used
     if (more) cp_async_wait<1>(); else cp_async_wait<0>();
     __syncthreads();                                             // tile `it` is complete and visible to every warp
-    const uint32_t ks = smem_u32(smem_raw + (it & 1) * kStage), vs = ks + kTileN * KP;
+    const uint32_t ks = smem_u32(smem_raw + (it & 1) * kStage), vs = SHARED ? ks : ks + kTileN * KP;
     // the barrier at the END of the body keeps stage it & 1 intact until every warp is done with it
     if (k0 > warp_last || (k0 + kTileN <= warp_first && k0 >= keep_hi)) { __syncthreads(); continue; }
     float sc[kTileN / 8][4];
@@ -343,23 +408,32 @@ __global__ void __launch_bounds__(128) sink_attention_mma_kernel(AttnArgs a) {
       const uint32_t a0 = ks + ((mj >> 1) * 8 + r) * KP + (mj & 1) * 16;
 #pragma unroll
       for (int kk = 0; kk < DP / 16; ++kk) {
+        uint32_t qa[4];
+        if constexpr (QS) {
+          ldmatrix_x4(qa, smem_u32(smem_raw + Tile::kQ) + (warp * 16 + (lane & 15)) * KP + kk * 32 + (lane >> 4) * 16);
+        } else {
+#pragma unroll
+          for (int e = 0; e < 4; ++e) qa[e] = qf[kk][e];
+        }
 #pragma unroll
         for (int jp = 0; jp < kTileN / 16; ++jp) {
           uint32_t bf[4];
           ldmatrix_x4(bf, a0 + jp * 16 * KP + kk * 32);
-          mma_m16n8k16<T>(sc[2 * jp], qf[kk], bf[0], bf[1]);
-          mma_m16n8k16<T>(sc[2 * jp + 1], qf[kk], bf[2], bf[3]);
+          mma_m16n8k16<T>(sc[2 * jp], qa, bf[0], bf[1]);
+          mma_m16n8k16<T>(sc[2 * jp + 1], qa, bf[2], bf[3]);
         }
       }
     }
     float mx[2] = {-INFINITY, -INFINITY};
 #pragma unroll
     for (int j = 0; j < kTileN / 8; ++j) {
+      float2 kf = make_float2(1.f, 1.f);
+      if (has_factor) kf = *reinterpret_cast<const float2*>(factors + (it & 1) * kTileN + j * 8 + 2 * tq);
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const int key = k0 + j * 8 + 2 * tq + (e & 1);
         const int lim = (e >> 1) ? pos1 : pos0, first = (e >> 1) ? lo1 : lo0;
-        float v = sc[j][e] * a.scale;
+        float v = sc[j][e] * a.scale * ((e & 1) ? kf.y : kf.x);
         if (cap > 0.f) v = cap * tanh_fast(v * inv_cap);
         v = (key <= lim && (key >= first || key < keep_hi)) ? v * kLog2e : -INFINITY;
         sc[j][e] = v;
@@ -446,55 +520,75 @@ __global__ void __launch_bounds__(128) sink_attention_mma_kernel(AttnArgs a) {
       den = l_run[r2] * num + fast_exp2(sk - mf);
     }
     inv[r2] = num / den;
-    if (a.gate && (r2 ? ok1 : ok0))
+    if (a.gate && !a.gate_elements && (r2 ? ok1 : ok0))
       inv[r2] *= gate_of(to_f32(((const T*)a.gate)[(int64_t)(start + t0 + (r2 ? r1 : r0)) * a.gate_stride + h]));
   }
   T* ob = (T*)a.out + h * Dv;
-  if (ok0) {
-    T* orow = ob + (int64_t)(start + t0 + r0) * a.out_stride;
+#pragma unroll
+  for (int r2 = 0; r2 < 2; ++r2) {
+    if (!(r2 ? ok1 : ok0)) continue;
+    const int64_t row = start + t0 + (r2 ? r1 : r0);
+    T* orow = ob + row * a.out_stride;
+    if (a.gate_elements) {                                       // all logits of the row in flight before the first store
+      const T* grow = (const T*)a.gate + row * a.gate_stride + h * Dv;
+      constexpr int B = DVP / 8 < 16 ? DVP / 8 : 16;
+#pragma unroll
+      for (int i0 = 0; i0 < DVP / 8; i0 += B) {
+        uint32_t gz[B];
+#pragma unroll
+        for (int i = 0; i < B; ++i)
+          gz[i] = (i0 + i) * 8 + 2 * tq < Dv ? *reinterpret_cast<const uint32_t*>(grow + (i0 + i) * 8 + 2 * tq) : 0u;
+#pragma unroll
+        for (int i = 0; i < B; ++i) {
+          const T* e = reinterpret_cast<const T*>(&gz[i]);
+          o[i0 + i][2 * r2] *= gate_of(to_f32(e[0]));
+          o[i0 + i][2 * r2 + 1] *= gate_of(to_f32(e[1]));
+        }
+      }
+    }
 #pragma unroll
     for (int i = 0; i < DVP / 8; ++i)
-      if (i * 8 + 2 * tq < Dv) *reinterpret_cast<uint32_t*>(orow + i * 8 + 2 * tq) = pack2<T>(o[i][0] * inv[0], o[i][1] * inv[0]);
-  }
-  if (ok1) {
-    T* orow = ob + (int64_t)(start + t0 + r1) * a.out_stride;
-#pragma unroll
-    for (int i = 0; i < DVP / 8; ++i)
-      if (i * 8 + 2 * tq < Dv) *reinterpret_cast<uint32_t*>(orow + i * 8 + 2 * tq) = pack2<T>(o[i][2] * inv[1], o[i][3] * inv[1]);
+      if (i * 8 + 2 * tq < Dv)
+        *reinterpret_cast<uint32_t*>(orow + i * 8 + 2 * tq) = pack2<T>(o[i][2 * r2] * inv[r2], o[i][2 * r2 + 1] * inv[r2]);
   }
 }
 
-template <typename T, int DP, int DVP>
+template <typename T, int DP, int DVP, bool SHARED>
 int launch_attention_mma(const AttnArgs& a, int max_q_len, int64_t num_seqs, cudaStream_t st) {
-  constexpr int smem = 2 * kTileN * ((DP + 8) * 2 + (DVP + 8) * 2);      // two stages
+  constexpr int smem = MmaTile<DP, DVP, SHARED>::kBytes;
   static int cache[64] = {0};
-  B2L_CUDA_CHECK(b2l_ensure_dynamic_smem(sink_attention_mma_kernel<T, DP, DVP>, smem, cache));
+  B2L_CUDA_CHECK(b2l_ensure_dynamic_smem(sink_attention_mma_kernel<T, DP, DVP, SHARED>, smem, cache));
   const int per = a.H / a.G;
   const dim3 grid = a.head_rows ? dim3((unsigned)a.nsplit, (unsigned)(a.G * ((per + kTileM - 1) / kTileM)), (unsigned)num_seqs)
                                 : dim3((unsigned)((max_q_len + kTileM - 1) / kTileM), (unsigned)a.H, (unsigned)num_seqs);
-  b2l_launch(sink_attention_mma_kernel<T, DP, DVP>, grid, dim3(128), (size_t)smem, st, a);
+  b2l_launch(sink_attention_mma_kernel<T, DP, DVP, SHARED>, grid, dim3(128), (size_t)smem, st, a);
   B2L_LAUNCH_CHECK();
   return B2L_OK;
 }
 
 template <typename T>
 int dispatch_attention_mma(const AttnArgs& a, int max_q_len, int64_t num_seqs, cudaStream_t st) {
-  const int dp = a.D <= 32 ? 32 : (a.D <= 64 ? 64 : 128), dvp = a.Dv <= 32 ? 32 : (a.Dv <= 64 ? 64 : 128);
-#define B2L_MMA(P, V) if (dp == P && dvp == V) return launch_attention_mma<T, P, V>(a, max_q_len, num_seqs, st)
-  B2L_MMA(32, 32); B2L_MMA(32, 64); B2L_MMA(32, 128);
-  B2L_MMA(64, 32); B2L_MMA(64, 64); B2L_MMA(64, 128);
-  B2L_MMA(128, 32); B2L_MMA(128, 64); B2L_MMA(128, 128);
+#define B2L_MMA(P, V, S) if (a.D <= P && a.Dv <= V) return launch_attention_mma<T, P, V, S>(a, max_q_len, num_seqs, st)
+  if (a.shared) {                                // smallest tile first
+    B2L_MMA(32, 32, true); B2L_MMA(64, 64, true); B2L_MMA(128, 128, true); B2L_MMA(160, 128, true);
+    B2L_MMA(192, 128, true); B2L_MMA(256, 128, true); B2L_MMA(256, 256, true); B2L_MMA(320, 256, true);
+  } else {
+    B2L_MMA(32, 32, false); B2L_MMA(32, 64, false); B2L_MMA(32, 128, false);
+    B2L_MMA(64, 32, false); B2L_MMA(64, 64, false); B2L_MMA(64, 128, false);
+    B2L_MMA(128, 32, false); B2L_MMA(128, 64, false); B2L_MMA(128, 128, false);
+  }
 #undef B2L_MMA
   B2L_UNSUPPORTED("sink_attention: head sizes %d / %d", a.D, a.Dv);
 }
 
-// the tensor-core tiled kernel takes 16-bit activations, head sizes in 8-element steps up to 128, and pool / q rows
-// whose 16-byte vectors are aligned
+// the tensor-core tiled kernel takes 16-bit activations, head sizes in 8-element steps up to 128 (values inside the
+// keys: up to 320 / 256), and pool / q / gate rows whose vectors are aligned
 inline bool mma_path_ok(const AttnArgs& a, int dtype) {
   if (dtype != B2L_F16 && dtype != B2L_BF16) return false;
-  if (a.D % 8 || a.Dv % 8 || a.D > 128 || a.Dv > 128) return false;
+  if (a.D % 8 || a.Dv % 8 || a.D > (a.shared ? 320 : 128) || a.Dv > (a.shared ? 256 : 128)) return false;
   if (a.kv_stride % 8 || a.v_col0 % 8 || a.v_hstride % 8 || a.q_stride % 2 || a.out_stride % 2) return false;
   if (((uintptr_t)a.kv % 16) || ((uintptr_t)a.q % 4) || ((uintptr_t)a.out % 4)) return false;
+  if (a.gate_elements && (a.gate_stride % 2 || ((uintptr_t)a.gate % 4))) return false;
   return true;
 }
 
@@ -513,13 +607,15 @@ __global__ void __launch_bounds__(128) sink_attention_split_kernel(AttnArgs a) {
   extern __shared__ __align__(16) uint8_t smem_raw[];
   const int D = a.D, Dv = a.Dv, per = a.H / a.G;
   constexpr int VEC = 16 / (int)sizeof(T);
-  const int Dp = (D + VEC - 1) / VEC * VEC + VEC, Dvp = (Dv + VEC - 1) / VEC * VEC;       // stage pitches (elements)
+  // stage pitches (elements); values inside the keys are read from the keys' stage
+  const int Dp = (D + VEC - 1) / VEC * VEC + VEC, Dvp = a.shared ? 0 : (Dv + VEC - 1) / VEC * VEC;
+  const int vp = a.shared ? Dp : Dvp;
   float* qs = reinterpret_cast<float*>(smem_raw);                        // [kSplitRows][D]
   float* mrg = qs + kSplitRows * ((D + 3) / 4 * 4);                      // [4 warps][kSplitRows][2 + Dv]
   T* stage = reinterpret_cast<T*>(mrg + 4 * kSplitRows * (2 + Dv) + ((4 - (4 * kSplitRows * (2 + Dv)) % 4) % 4));
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   T* ks = stage + (size_t)warp * 32 * (Dp + Dvp);
-  T* vs = ks + 32 * Dp;
+  T* vs = a.shared ? ks : ks + 32 * Dp;
   const int z = blockIdx.z, s = a.seq_list ? a.seq_list[z] : z;
   const int start = a.seq_start[s], ctx = a.seq_ctx[s];
   const int64_t slot = a.seq_slot[s];
@@ -551,6 +647,8 @@ __global__ void __launch_bounds__(128) sink_attention_split_kernel(AttnArgs a) {
                       (a.v_hstride % VEC == 0) && (((uintptr_t)a.kv % 16) == 0);
   for (int k0 = key_lo + warp * 32; k0 < key_hi; k0 += 128) {
     const int nk = min(32, key_hi - k0);
+    float factor = a.scale;                        // lane j: what multiplies key j's dot products
+    if (a.key_factor_col >= 0 && lane < nk) factor *= key_factor<T>(a, trow[axis.key(k0 + lane)]);
     __syncwarp();
     if (vec_ok) {
       // lane j fetches key j's pool row once; the 16-byte copies run in batches of kStageBatch loads per lane that
@@ -574,13 +672,13 @@ __global__ void __launch_bounds__(128) sink_attention_split_kernel(AttnArgs a) {
         }
       };
       stage_rows(ks, Dp, g * D, D / VEC);
-      stage_rows(vs, Dvp, v_col, Dv / VEC);
+      if (!a.shared) stage_rows(vs, Dvp, v_col, Dv / VEC);
     } else {
       for (int i = lane; i < nk * D; i += 32) {
         const int j = i / D, d = i - j * D;
         ks[j * Dp + d] = kv[(int64_t)trow[axis.key(k0 + j)] * a.kv_stride + g * D + d];
       }
-      for (int i = lane; i < nk * Dv; i += 32) {
+      for (int i = a.shared ? nk * Dv : lane; i < nk * Dv; i += 32) {
         const int j = i / Dv, d = i - j * Dv;
         vs[j * Dvp + d] = kv[(int64_t)trow[axis.key(k0 + j)] * a.kv_stride + v_col + d];
       }
@@ -613,7 +711,7 @@ __global__ void __launch_bounds__(128) sink_attention_split_kernel(AttnArgs a) {
 #pragma unroll
     for (int r = 0; r < kSplitRows; ++r) {
       if (r >= h_count) continue;
-      float sv = sc[r] * a.scale;
+      float sv = sc[r] * factor;
       if (a.softcap > 0.f) sv = a.softcap * tanhf(sv * inv_cap);
       const bool ok = lane < nk;
       sv = ok ? sv : -INFINITY;
@@ -631,7 +729,7 @@ __global__ void __launch_bounds__(128) sink_attention_split_kernel(AttnArgs a) {
 #pragma unroll
       for (int j = 0; j < DVJ; ++j) {
         const int d = lane + 32 * j;
-        vv[j] = d < Dv ? to_f32(vs[kk * Dvp + d]) : 0.f;
+        vv[j] = d < Dv ? to_f32(vs[kk * vp + d]) : 0.f;
       }
 #pragma unroll
       for (int r = 0; r < kSplitRows; ++r) {
@@ -676,7 +774,7 @@ __global__ void __launch_bounds__(128) sink_attention_split_kernel(AttnArgs a) {
 template <typename T>
 int launch_attention_split(const AttnArgs& a, int64_t num_seqs, cudaStream_t st) {
   constexpr int VEC = 16 / (int)sizeof(T);
-  const int Dp = (a.D + VEC - 1) / VEC * VEC + VEC, Dvp = (a.Dv + VEC - 1) / VEC * VEC;
+  const int Dp = (a.D + VEC - 1) / VEC * VEC + VEC, Dvp = a.shared ? 0 : (a.Dv + VEC - 1) / VEC * VEC;
   const int Dq = (a.D + 3) / 4 * 4;
   int mfl = 4 * kSplitRows * (2 + a.Dv);
   mfl += (4 - mfl % 4) % 4;
@@ -712,7 +810,8 @@ __global__ void __launch_bounds__(64) sink_attention_merge_kernel(T* __restrict_
                                                                   const int* __restrict__ seq_start,
                                                                   const int* __restrict__ seq_list, int H, int Dv,
                                                                   int nsplit, int sink_heads,
-                                                                  const T* __restrict__ gate, int64_t gate_stride) {
+                                                                  const T* __restrict__ gate, int64_t gate_stride,
+                                                                  int gate_elements) {
   pdl_prologue();
   __shared__ float wsm[kMergeCached];
   __shared__ float red[2];
@@ -740,13 +839,15 @@ __global__ void __launch_bounds__(64) sink_attention_merge_kernel(T* __restrict_
   if (sink) den += expf(to_f32(sink[h % sink_heads]) - mf);
   T* o = out + (int64_t)seq_start[s] * out_stride + h * Dv;
   float num = 1.0f;
-  if (gate) num = gate_of(to_f32(gate[(int64_t)seq_start[s] * gate_stride + h % sink_heads]));
+  const T* gr = gate ? gate + (int64_t)seq_start[s] * gate_stride : nullptr;
+  if (gr && !gate_elements) num = gate_of(to_f32(gr[h % sink_heads]));
   for (int d = tid; d < Dv; d += 64) {
     float v = 0.f;
     for (int i = 0; i < nsplit; ++i) {
       const float w = i < kMergeCached ? wsm[i] : expf(p[i * (Dv + 2)] - mf);
       v = fmaf(p[i * (Dv + 2) + 2 + d], w, v);
     }
+    if (gate_elements) num = gate_of(to_f32(gr[(h % sink_heads) * Dv + d]));
     o[d] = from_f32<T>(gate ? v / den * num : v / den);
   }
 }
@@ -1071,9 +1172,91 @@ __global__ void __launch_bounds__(256) attn_prepare_vec_kernel(
   }
 }
 
+// Keys that are values too: the row keeps the keys AS PROJECTED, and what the key norm would do to them goes elsewhere.
+// Its statistic (one per token) becomes the row's score factor; its channel weights, like the query norm's, multiply the
+// query (`w` [H * D] fp32 = query weight * weight of the key channel the query entry meets).
+//   q <- q / rms(q) * w * gain(position) in place;   pool row = [k as it is | 1 / rms(k) as fp32]
+// One CTA per token; both statistics in one block reduction.  V > 1: rows in 16-byte vectors, kept in registers (q up to
+// 2, k one vector per thread); V = 1: any size, read twice.
+template <typename T, int V>
+__global__ void __launch_bounds__(256) norm_query_keep_key_kernel(
+    T* __restrict__ qk, int64_t stride, T* __restrict__ kv, int64_t kv_stride, const int* __restrict__ rows,
+    const int* __restrict__ pos, const float* __restrict__ w, int qn, int kn, int factor_col, float eps, float gain_coef,
+    double gain_every) {
+  pdl_prologue();
+  __shared__ float red[16];
+  const int64_t t = blockIdx.x;
+  T* q = qk + t * stride;
+  const T* k = q + qn;
+  T* dst = kv + (int64_t)rows[t] * kv_stride;
+  float gain = 1.f;
+  if (gain_every > 0.0) gain = 1.0f + gain_coef * logf((float)floor(((double)pos[t] + 1.0) / gain_every) + 1.0f);
+  float sq = 0.f, sk = 0.f;
+  uint4 rq[kPrepQ], rk;
+  if constexpr (V > 1) {
+#pragma unroll
+    for (int u = 0; u < kPrepQ; ++u) {
+      const int i = (threadIdx.x + u * 256) * V;
+      rq[u] = make_uint4(0u, 0u, 0u, 0u);
+      if (i < qn) rq[u] = *reinterpret_cast<const uint4*>(q + i);
+    }
+    rk = make_uint4(0u, 0u, 0u, 0u);
+    if ((int)threadIdx.x * V < kn) rk = *reinterpret_cast<const uint4*>(k + threadIdx.x * V);
+#pragma unroll
+    for (int u = 0; u < kPrepQ; ++u) {
+      const T* e = reinterpret_cast<const T*>(&rq[u]);
+#pragma unroll
+      for (int c = 0; c < V; ++c) { const float x = to_f32(e[c]); sq = fmaf(x, x, sq); }
+    }
+    const T* e = reinterpret_cast<const T*>(&rk);
+#pragma unroll
+    for (int c = 0; c < V; ++c) { const float x = to_f32(e[c]); sk = fmaf(x, x, sk); }
+    if ((int)threadIdx.x * V < kn) *reinterpret_cast<uint4*>(dst + threadIdx.x * V) = rk;
+  } else {
+    for (int i = threadIdx.x; i < qn; i += 256) { const float x = to_f32(q[i]); sq = fmaf(x, x, sq); }
+    for (int i = threadIdx.x; i < kn; i += 256) {
+      const T raw = k[i];
+      const float x = to_f32(raw);
+      sk = fmaf(x, x, sk);
+      dst[i] = raw;
+    }
+  }
+  sq = warp_reduce_sum(sq);
+  sk = warp_reduce_sum(sk);
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  if (lane == 0) { red[warp] = sq; red[8 + warp] = sk; }
+  __syncthreads();
+  sq = sk = 0.f;
+#pragma unroll
+  for (int i = 0; i < 8; ++i) { sq += red[i]; sk += red[8 + i]; }
+  if (threadIdx.x == 0) *reinterpret_cast<float*>(dst + factor_col) = 1.0f / sqrtf(sk / (float)kn + eps);
+  const float f = gain / sqrtf(sq / (float)qn + eps);
+  if constexpr (V > 1) {
+#pragma unroll
+    for (int u = 0; u < kPrepQ; ++u) {
+      const int i = (threadIdx.x + u * 256) * V;
+      if (i >= qn) continue;
+      const T* e = reinterpret_cast<const T*>(&rq[u]);
+      uint4 res;
+      T* re = reinterpret_cast<T*>(&res);
+#pragma unroll
+      for (int c4 = 0; c4 < V; c4 += 4) {
+        const float4 wv = *reinterpret_cast<const float4*>(w + i + c4);
+        re[c4] = from_f32<T>(to_f32(e[c4]) * f * wv.x);
+        re[c4 + 1] = from_f32<T>(to_f32(e[c4 + 1]) * f * wv.y);
+        re[c4 + 2] = from_f32<T>(to_f32(e[c4 + 2]) * f * wv.z);
+        re[c4 + 3] = from_f32<T>(to_f32(e[c4 + 3]) * f * wv.w);
+      }
+      *reinterpret_cast<uint4*>(q + i) = res;
+    }
+  } else {
+    for (int i = threadIdx.x; i < qn; i += 256) q[i] = from_f32<T>(to_f32(q[i]) * f * w[i]);
+  }
+}
+
 template <typename T>
 int launch_attention(const AttnArgs& a, dim3 grid, cudaStream_t st) {
-  const size_t smem = (size_t)(kRows * a.D + kKeys * (a.D + 1) + kKeys * a.Dv) * sizeof(float);
+  const size_t smem = (size_t)(kRows * a.D + kKeys * (a.D + 2) + (a.shared ? 0 : kKeys * a.Dv)) * sizeof(float);
   B2L_REQUIRE((int64_t)smem <= b2l_max_smem_optin(), "sink_attention: head sizes %d / %d need %lld bytes of shared memory",
               a.D, a.Dv, (long long)smem);
   const int dvj = (a.Dv + 31) / 32;
@@ -1124,6 +1307,33 @@ extern "C" int b2l_attn_prepare(void* qkv, int64_t qkv_row_stride, void* kv_pool
   return B2L_OK;
 }
 
+extern "C" int b2l_norm_query_keep_key(void* qk, int64_t qk_row_stride, void* kv_pool, int64_t kv_row_stride,
+                                       const void* kv_rows_i32, const void* pos_i32, const void* query_weight_f32,
+                                       int64_t tokens, int q_cols, int k_cols, int factor_col, float eps,
+                                       float gain_coef, float gain_every, int dtype, void* stream) {
+  B2L_REQUIRE(qk && kv_pool && kv_rows_i32 && pos_i32 && query_weight_f32, "norm_query_keep_key: null pointer");
+  B2L_REQUIRE(q_cols > 0 && k_cols > 0 && factor_col >= k_cols, "norm_query_keep_key: bad shape");
+  B2L_REQUIRE(dtype == B2L_F32 || (factor_col % 2 == 0 && kv_row_stride % 2 == 0 && (uintptr_t)kv_pool % 4 == 0),
+              "norm_query_keep_key: the score factors must be 4-byte aligned");
+  if (tokens <= 0) return B2L_OK;
+  cudaStream_t st = (cudaStream_t)stream;
+  B2L_DISPATCH_FLOAT(dtype, "norm_query_keep_key", {
+    constexpr int VEC = 16 / (int)sizeof(T);
+    auto al = [](const void* p) { return (uintptr_t)p % 16 == 0; };
+    const bool vec = q_cols % VEC == 0 && k_cols % VEC == 0 && qk_row_stride % VEC == 0 && kv_row_stride % VEC == 0 &&
+                     q_cols <= kPrepQ * 256 * VEC && k_cols <= 256 * VEC && al(qk) && al(kv_pool) && al(query_weight_f32);
+    auto go = [&](auto kernel) {
+      b2l_launch(kernel, dim3((unsigned)tokens), dim3(256), (size_t)0, st, (T*)qk, qk_row_stride, (T*)kv_pool, kv_row_stride,
+                 (const int*)kv_rows_i32, (const int*)pos_i32, (const float*)query_weight_f32, q_cols, k_cols, factor_col,
+                 eps, gain_coef, (double)gain_every);
+    };
+    if (vec) go(norm_query_keep_key_kernel<T, VEC>);
+    else go(norm_query_keep_key_kernel<T, 1>);
+  });
+  B2L_LAUNCH_CHECK();
+  return B2L_OK;
+}
+
 extern "C" int64_t b2l_sink_attention_workspace_bytes(int64_t num_seqs, int heads, int v_head_dim, int num_splits) {
   if (num_splits <= 0) return 0;
   return num_seqs * heads * (int64_t)num_splits * (v_head_dim + 2) * 4;
@@ -1133,7 +1343,8 @@ extern "C" int64_t b2l_sink_attention_workspace_bytes(int64_t num_seqs, int head
  * and `split_keys` keys go to each of the num_splits ranges, counted from the token's first visible key
  * (num_splits * split_keys >= the most keys any listed token sees: context + 1, or window + keep_first if that is
  * smaller).  window <= 0: no sliding window; keep_first (with a window): the first positions that stay visible;
- * gate (nullable) [tokens, >= heads]: head h's output times sigmoid(gate[t, h]); block > 0 (window <= 0): block-diagonal mask; v_col0 < 0: the values follow the keys in a pool row (column kv_heads * head_dim);
+ * gate (nullable) [tokens, >= heads]: head h's output times sigmoid(gate[t, h]) (gate_elements: [tokens, heads *
+ * v_head_dim], element by element); key_factor_col >= 0: the column of a pool row's fp32 score factor; block > 0 (window <= 0): block-diagonal mask; v_col0 < 0: the values follow the keys in a pool row (column kv_heads * head_dim);
  * v_head_stride < 0: kv head g's values start g * v_head_dim columns after v_col0 (0: all kv heads read the same columns).
  * v_blocks > 1 (split mode): block c of v_head_dim value columns starts c * v_head_dim columns further and is one more
  * set of `heads` results, out [v_blocks][heads][v_head_dim] per token, in the same two launches (workspace for
@@ -1144,8 +1355,8 @@ extern "C" int b2l_sink_attention(void* out, int64_t out_row_stride, const void*
                                   const void* seq_slot, const void* seq_list, int64_t num_seqs, int max_q_len,
                                   const void* sink, int heads, int kv_heads, int head_dim, int v_head_dim, float scale,
                                   float softcap, int window, int keep_first, int block, int v_col0, int v_head_stride,
-                                  int v_blocks, const void* gate, int64_t gate_row_stride, int num_splits,
-                                  int split_keys, void* workspace, int64_t workspace_bytes, int dtype, void* stream) {
+                                  int v_blocks, const void* gate, int64_t gate_row_stride, int gate_elements,
+                                  int key_factor_col, int num_splits, int split_keys, void* workspace, int64_t workspace_bytes, int dtype, void* stream) {
   B2L_REQUIRE(out && q && kv_pool && table_i32 && seq_start && seq_ctx && seq_slot, "sink_attention: null pointer");
   B2L_REQUIRE(heads > 0 && kv_heads > 0 && heads % kv_heads == 0, "sink_attention: %d heads must be a multiple of num_kv_heads %d",
               heads, kv_heads);
@@ -1166,11 +1377,16 @@ extern "C" int b2l_sink_attention(void* out, int64_t out_row_stride, const void*
   a.window = window > 0 ? window : 0;
   a.block = (window <= 0 && block > 0) ? block : 0;
   a.keep = (window > 0 && keep_first > 0) ? keep_first : 0;
-  a.gate = gate; a.gate_stride = gate_row_stride;
+  a.gate = gate; a.gate_stride = gate_row_stride; a.gate_elements = gate ? gate_elements : 0;
+  a.key_factor_col = key_factor_col;
+  B2L_REQUIRE(key_factor_col < 0 || (dtype == B2L_F32 ? true : key_factor_col % 2 == 0 && kv_row_stride % 2 == 0),
+              "sink_attention: the score factors must be 4-byte aligned");
   a.v_col0 = v_col0 >= 0 ? v_col0 : kv_heads * head_dim;
   a.v_hstride = v_head_stride >= 0 ? v_head_stride : v_head_dim;
   a.head_rows = 0;
   a.v_blocks = v_blocks > 1 ? v_blocks : 1;
+  a.shared = a.v_col0 == 0 && v_head_dim <= head_dim && a.v_blocks == 1 && (kv_heads == 1 || a.v_hstride == head_dim);
+  B2L_REQUIRE(!a.gate_elements || a.v_blocks == 1, "sink_attention: one value block with an element gate");
   B2L_REQUIRE(a.v_blocks == 1 || num_splits > 0, "sink_attention: value blocks are for steps of single tokens");
   const int hchunks = (per + a.PH - 1) / a.PH;
   if (num_splits > 0) {
@@ -1194,7 +1410,7 @@ extern "C" int b2l_sink_attention(void* out, int64_t out_row_stride, const void*
       b2l_launch(sink_attention_merge_kernel<T>, dim3((unsigned)(heads * a.v_blocks), (unsigned)num_seqs), dim3(64),
                  (size_t)0, st, (T*)out, out_row_stride, (const float*)workspace, (const T*)sink,
                  (const int*)seq_start, (const int*)seq_list, heads * a.v_blocks, v_head_dim, num_splits, heads,
-                 (const T*)gate, gate_row_stride);
+                 (const T*)gate, gate_row_stride, a.gate_elements);
     });
     B2L_LAUNCH_CHECK();
     return B2L_OK;
@@ -1243,6 +1459,7 @@ extern "C" int b2l_mixed_head_attention(void* out, int64_t out_row_stride, const
   a.v_col0 = v_col0 >= 0 ? v_col0 : kv_heads * head_dim;
   a.v_hstride = v_head_dim;
   a.v_blocks = 1;
+  a.key_factor_col = -1;
   cudaStream_t st = (cudaStream_t)stream;
   int rc = B2L_OK;
   B2L_DISPATCH_FLOAT(dtype, "mixed_head_attention", { rc = launch_mixed_head_attention<T>(a, mix, num_seqs, st); });

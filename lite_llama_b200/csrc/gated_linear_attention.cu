@@ -27,7 +27,7 @@
 //                    (sum_j (sum_g M[h,g] p_g(j)) v(j) = sum_g M[h,g] (sum_j p_g(j) v(j)))
 //   swiglu_scaled    out[r, :] = silu(s_r * gate) * (s_r * up) * sigmoid(z_r): a gated activation whose INPUT carries
 //                    a per-row fp32 factor (an expert weight on the expert's input: W (s x) = s (W x)) and whose output
-//                    a per-row logistic gate (both optional); the unit may be the clamped form of gated_unit.cuh instead
+//                    a per-row logistic gate (both optional); the unit may be another form of gated_unit.cuh instead
 #include "common.cuh"
 #include "gated_unit.cuh"
 #include "rowvec.cuh"
@@ -550,7 +550,7 @@ extern "C" int b2l_swiglu_scaled(void* out, int64_t out_row_stride, const void* 
                                  int64_t z_row_stride, int64_t rows, int64_t n, int form, float limit, float alpha,
                                  int dtype, void* stream) {
   B2L_REQUIRE(out && gate && up, "swiglu_scaled: null pointer");
-  B2L_REQUIRE(n > 0 && (form == kUnitSilu || form == kUnitClamped), "swiglu_scaled: bad shape or form %d", form);
+  B2L_REQUIRE(n > 0 && form >= kUnitSilu && form <= kUnitGeluTanh, "swiglu_scaled: bad shape or form %d", form);
   const GatedUnit unit{form, limit, alpha};
   if (rows <= 0) return B2L_OK;
   cudaStream_t st = (cudaStream_t)stream;

@@ -4,7 +4,8 @@
 // the latent itself):
 //
 //   proj row  = [ a: q_rank | b: kv_rank | r: rot_dim | ... ]          (one fused down-projection of the mixer input)
-//   a  <- a / rms(a) * wq                in place: the input of the query up-projection
+//   a  <- a / rms(a) * wq                in place: the input of the query up-projection (q_rank 0: queries are projected
+//                                        from the mixer input directly, there is no a)
 //   pool row  = [ b / rms(b) * wkv | rotate(r, pos) ]
 //
 //   rope_heads: dst[t, h, :width] = src[t, h, :width] with the first `rot_dims` entries rotated by the token's position;
@@ -58,10 +59,12 @@ __global__ void __launch_bounds__(128) latent_prepare_kernel(T* __restrict__ pro
   const T* b = a + q_rank;
   const T* r = b + kv_rank;
   T* dst = pool + (int64_t)rows[t] * pool_stride;
-  float ss = 0.f;
-  for (int i = lane; i < q_rank; i += 32) { const float v = to_f32(a[i]); ss = fmaf(v, v, ss); }
-  float rstd = 1.0f / sqrtf(warp_reduce_sum(ss) / (float)q_rank + eps);
-  for (int i = lane; i < q_rank; i += 32) a[i] = from_f32<T>(to_f32(a[i]) * rstd * to_f32(wq[i]));
+  float ss = 0.f, rstd;
+  if (q_rank > 0) {
+    for (int i = lane; i < q_rank; i += 32) { const float v = to_f32(a[i]); ss = fmaf(v, v, ss); }
+    rstd = 1.0f / sqrtf(warp_reduce_sum(ss) / (float)q_rank + eps);
+    for (int i = lane; i < q_rank; i += 32) a[i] = from_f32<T>(to_f32(a[i]) * rstd * to_f32(wq[i]));
+  }
   ss = 0.f;
   for (int i = lane; i < kv_rank; i += 32) { const float v = to_f32(b[i]); ss = fmaf(v, v, ss); }
   rstd = 1.0f / sqrtf(warp_reduce_sum(ss) / (float)kv_rank + eps);
@@ -125,8 +128,8 @@ extern "C" int b2l_latent_prepare(void* proj, int64_t proj_row_stride, void* poo
                                   const void* kv_rows_i32, const void* cos_sin_f32, const void* q_norm_weight,
                                   const void* kv_norm_weight, int64_t tokens, int q_rank, int kv_rank, int rot_dim,
                                   int rot_dims, int pairing, float eps, int dtype, void* stream) {
-  B2L_REQUIRE(proj && pool && kv_rows_i32 && q_norm_weight && kv_norm_weight, "latent_prepare: null pointer");
-  B2L_REQUIRE(q_rank > 0 && kv_rank > 0 && rot_dim >= 0 && rot_dims >= 0 && rot_dims <= rot_dim && rot_dims % 2 == 0,
+  B2L_REQUIRE(proj && pool && kv_rows_i32 && (q_norm_weight || q_rank == 0) && kv_norm_weight, "latent_prepare: null pointer");
+  B2L_REQUIRE(q_rank >= 0 && kv_rank > 0 && rot_dim >= 0 && rot_dims >= 0 && rot_dims <= rot_dim && rot_dims % 2 == 0,
               "latent_prepare: bad shape (q_rank %d, kv_rank %d, rot_dim %d, rot_dims %d)", q_rank, kv_rank, rot_dim, rot_dims);
   B2L_REQUIRE(cos_sin_f32 || rot_dims == 0, "latent_prepare: no rotation table");
   if (tokens <= 0) return B2L_OK;

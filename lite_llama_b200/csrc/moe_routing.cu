@@ -143,14 +143,15 @@ __global__ void moe_route_kernel(const T* __restrict__ logits, int64_t row_strid
 // Router with a selection bias and group-limited choice (one CTA per token; the router product is done here,
 // or comes as fp32 logits from a GEMM, in which case the CTA is a single warp):
 //   z = W_r . x (fp32 sums),  s = sigmoid(z), or softmax(z) over all experts (`softmax`),  choice = s + bias
-//   the experts form `groups` equal runs of neighbours; a group's score = the sum of its two largest choice scores;
+//   the experts form `groups` equal runs of neighbours; a group's score = the sum of its two largest choice scores
+//   (`group_best`: its largest alone);
 //   only experts of the `keep` best groups can be chosen; the `top_k` largest choice scores among them win
 //   (lowest index on ties); weights = scale * s of the winners / (their sum + 1e-20), fp32.
 template <typename T>
 __global__ void __launch_bounds__(128) moe_route_sigmoid_kernel(const T* __restrict__ x, int64_t xs,
                                                                 const T* __restrict__ wr, const T* __restrict__ bias,
                                                                 const float* __restrict__ logits, int num_experts,
-                                                                int k, int top_k, int groups, int keep,
+                                                                int k, int top_k, int groups, int keep, int group_best,
                                                                 int renormalize, int softmax, float scale,
                                                                 float* __restrict__ out_w,
                                                                 int* __restrict__ out_ids) {
@@ -202,7 +203,7 @@ __global__ void __launch_bounds__(128) moe_route_sigmoid_kernel(const T* __restr
       const float v = ch[e];
       if (v > a) { b = a; a = v; } else if (v > b) { b = v; }
     }
-    gs[g] = per > 1 ? a + b : a;
+    gs[g] = per > 1 && !group_best ? a + b : a;
   }
   __syncthreads();
   if (warp != 0) return;
@@ -316,12 +317,13 @@ extern "C" int b2l_moe_route_topk(void* topk_weights, void* topk_ids_i64, const 
 /* Sigmoid scores + selection bias + group-limited top-k (fp32 throughout).  The router product is done here from
  * x [tokens, k] and router_w [experts, k] in dtype, unless logits_f32 [tokens, experts] brings it; bias [experts] in
  * dtype (nullable); weights_f32 [tokens, top_k], ids_i32 [tokens, top_k].  groups must divide experts; keep <= groups.
+ * group_best: a group scores its largest choice score instead of the sum of its two largest.
  * renormalize 0: the weights are the winners' scores themselves, not divided by their sum.  softmax: the scores are the
  * softmax over all experts instead of sigmoids.  scale multiplies the weights. */
 extern "C" int b2l_moe_route_sigmoid_groups(void* weights_f32, void* ids_i32, const void* x, int64_t x_row_stride,
                                             const void* router_w, const void* bias, const void* logits_f32,
                                             int64_t tokens, int num_experts, int64_t k, int top_k, int groups, int keep,
-                                            int renormalize, int softmax, float scale, int dtype, void* stream) {
+                                            int group_best, int renormalize, int softmax, float scale, int dtype, void* stream) {
   B2L_REQUIRE(weights_f32 && ids_i32 && ((x && router_w) || logits_f32), "moe_route_sigmoid_groups: null pointer");
   B2L_REQUIRE(num_experts > 0 && k > 0 && k < (1ll << 31) && top_k >= 1 && top_k <= num_experts && groups >= 1 &&
                   num_experts % groups == 0 && keep >= 1 && keep <= groups &&
@@ -334,7 +336,7 @@ extern "C" int b2l_moe_route_sigmoid_groups(void* weights_f32, void* ids_i32, co
   B2L_DISPATCH_FLOAT(dtype, "moe_route_sigmoid_groups", {
     b2l_launch(moe_route_sigmoid_kernel<T>, dim3((unsigned)tokens), dim3(logits_f32 ? 32 : 128), smem, st, (const T*)x,
                x_row_stride, (const T*)router_w, (const T*)bias, (const float*)logits_f32, num_experts, (int)k, top_k,
-               groups, keep, renormalize, softmax, scale, (float*)weights_f32, (int*)ids_i32);
+               groups, keep, group_best, renormalize, softmax, scale, (float*)weights_f32, (int*)ids_i32);
   });
   B2L_LAUNCH_CHECK();
   return B2L_OK;

@@ -36,6 +36,9 @@ Designs registered here:
     memory with exponential gates, window attention with kept first tokens, sinks and head gates (some layers read
     another layer's cache), latent attention with an element-wise output gate; clamped gated experts behind a softmax
     router.
+  * ``Povilorn``: element-wise ``tanh`` norms in front of the sublayers, a loop over some of the layers (every pass with a
+    cache of its own); latent attention without a query latent and with interpolated rotary frequencies, position-free
+    attention whose values are its keys; clamped experts in groups, identity experts among them.
 """
 
 from __future__ import annotations
@@ -58,6 +61,8 @@ from ..kernels import (
     gelu,
     gelu_mul_gather,
     grouped_experts,
+    key_factor_column,
+    norm_query_keep_key,
     head_linear,
     head_mix,
     head_norm_gate,
@@ -83,6 +88,7 @@ from ..kernels import (
     stream_mix,
     swiglu_forward,
     swiglu_scaled,
+    tanh_norm_stream,
 )
 from .model_config import (BlockAttentionSpec, ConvWindowAttentionSpec, DecayAttentionSpec, DeltaRuleSpec, DenseMlpSpec,
                            ForgetGateAttentionSpec, LatentAttentionSpec, LayeredConfig, LayerSpec, Mamba2Spec,
@@ -106,7 +112,8 @@ class LayeredLayerWeights:
     side: dict[str, torch.Tensor] | None = None          # per-layer token input: gate, proj, norm
     depth: torch.Tensor | None = None                    # depth-average coefficients over [embedding, layer results]
     # stream designs, one dict per sublayer (mixer, feed-forward): read coefficients "in" [streams], write coefficients
-    # "coef" [out | mix] (both fp32), "norm", input convolution "conv", result gate "gate", "gate_b"
+    # "coef" [out | mix] (both fp32), "norm", input convolution "conv", result gate "gate", "gate_b"; tanh-norm designs:
+    # "norm", its shift "norm_b" and its "alpha"
     subs: list[dict[str, torch.Tensor]] | None = None
 
 
@@ -120,6 +127,8 @@ class LayeredWeights:
     embed_norm: torch.Tensor | None = None
     side_embed: torch.Tensor | None = None               # [vocab, layers * token_side_dim]
     stream_ones: torch.Tensor | None = None              # fp32 ones [streams]: the output reads the sum of the streams
+    final_sub: dict[str, torch.Tensor] | None = None     # tanh-norm designs: the output norm, as a layer's "subs" entry
+    loop_step: torch.Tensor | None = None                # [passes, hidden]: what each pass of a loop adds at its start
 
     def nbytes_per_step(self) -> int:
         """Weight bytes one step streams (embedding / position gathers excluded)."""
@@ -198,29 +207,39 @@ _MAX_SPLITS = 128
 
 def sink_attention_mixer(li: int, spec: SinkAttentionSpec, w: dict[str, torch.Tensor], x: torch.Tensor,
                          ctx: StepContext, eps: float) -> torch.Tensor:
-    """fused q|k|v projection -> per-token preparation (norms, query gain, value mixing, cache write) -> attention
-    over the pool: the tiled kernel for prompt portions, the key-split kernel for single tokens."""
+    """fused q|k|v (or q|k when the keys are the values) projection, output gate logits behind it -> per-token preparation
+    (norms, query gain, value mixing, cache write) -> attention over the pool, gated in its epilogue: the tiled kernel for
+    prompt portions, the key-split kernel for single tokens."""
     b = ctx.batch
     qn, kn, vn = spec.heads * spec.head_dim, spec.kv_heads * spec.head_dim, spec.kv_heads * spec.v_head_dim
-    qkv = linear(x, w["qkv"])
+    qkv = linear(x, w["qkv"], w.get("qkv_b"))
     pool = ctx.kv_buffer[li]
     v_in = v_out = None
-    if spec.v_mix:
+    form = {}
+    if spec.element_gate:
+        g0 = aligned_columns(qn + kn + (0 if spec.keys_as_values else vn), 0)[1]
+        form = dict(gate=qkv[:, g0:g0 + spec.heads * spec.v_head_dim], gate_elements=True)
+    if spec.keys_as_values:
+        norm_query_keep_key(qkv, pool, b.kv_rows, b.positions, qn, kn, w["query_weight"], eps, spec.gain_coef,
+                            spec.gain_every)
+        form.update(v_col0=0, v_head_stride=spec.head_dim, key_factor_col=key_factor_column(kn))
+    elif spec.v_mix:
         if ctx.v_first is None:
             ctx.v_first = v_out = torch.empty((b.tokens, vn), dtype=qkv.dtype, device=qkv.device)
         else:
             v_in = ctx.v_first
-    attn_prepare(qkv, pool, b.kv_rows, b.positions, qn, kn, vn, w.get("q_norm"), w.get("k_norm"), eps,
-                 spec.gain_coef, spec.gain_every, v_in, v_out, w.get("vmix") if v_in is not None else None)
+    if not spec.keys_as_values:
+        attn_prepare(qkv, pool, b.kv_rows, b.positions, qn, kn, vn, w.get("q_norm"), w.get("k_norm"), eps,
+                     spec.gain_coef, spec.gain_every, v_in, v_out, w.get("vmix") if v_in is not None else None)
     out = torch.empty((b.tokens, spec.heads * spec.v_head_dim), dtype=qkv.dtype, device=qkv.device)
     common = (spec.heads, spec.kv_heads, spec.head_dim, spec.v_head_dim, spec.scale, spec.softcap)
     if b.num_portions:
         sink_attention(out, qkv, pool, ctx.table, b.seq_start, b.seq_ctx, b.seq_slot, b.portion_list, b.num_portions,
-                       b.max_portion, w.get("sink"), *common)
+                       b.max_portion, w.get("sink"), *common, **form)
     if b.num_singles:
         splits, per = split_plan(b.max_single_ctx + 1)
         sink_attention(out, qkv, pool, ctx.table, b.seq_start, b.seq_ctx, b.seq_slot, b.single_list, b.num_singles, 1,
-                       w.get("sink"), *common, num_splits=splits, split_keys=per)
+                       w.get("sink"), *common, num_splits=splits, split_keys=per, **form)
     return linear(out, w["o"])
 
 
@@ -233,8 +252,8 @@ def split_plan(keys: int) -> tuple[int, int]:
 
 def latent_attention_mixer(li: int, spec: LatentAttentionSpec, w: dict[str, torch.Tensor], x: torch.Tensor,
                            ctx: StepContext, eps: float) -> torch.Tensor:
-    """One fused down-projection [query latent | key/value latent | shared rotated key part | head gates] -> latent
-    norms, rotation and the cache write (``latent_prepare``) -> query up-projection -> the queries' unrotated parts
+    """One fused down-projection [query latent | key/value latent | shared rotated key part | head gates] (no query latent:
+    the queries themselves in its place) -> latent norms, rotation and the cache write (``latent_prepare``) -> query up-projection -> the queries' unrotated parts
     multiplied into the latent space per head (``W_uk^T q``), their rotated parts turned by the position -> attention
     over the cached rows [latent | rotated key part] as ONE key/value head whose values are the latent itself (sliding
     window) -> per-head value up-projection with the sigmoid gate (one per head, or per element) in its epilogue ->
@@ -244,10 +263,17 @@ def latent_attention_mixer(li: int, spec: LatentAttentionSpec, w: dict[str, torc
     H, dim, rot, rank = spec.heads, spec.head_dim, spec.rot_dim, spec.kv_rank
     proj = linear(x, w["down"])
     pool = ctx.kv_buffer[li]
-    cos_sin = ctx.rope(spec.rot_dims, spec.rot_base)
-    latent_prepare(proj, pool, b.kv_rows, cos_sin, w["q_norm"], w["kv_norm"], spec.q_rank, rank, rot, spec.rot_dims, eps,
-                   spec.pairing)
-    q = linear(proj[:, :spec.q_rank], w["uq"])
+    cos_sin = ctx.rope_freqs(w["freqs"], spec_magnitude(spec)) if "freqs" in w else ctx.rope(spec.rot_dims, spec.rot_base)
+    if spec.q_rank:
+        latent_prepare(proj, pool, b.kv_rows, cos_sin, w["q_norm"], w["kv_norm"], spec.q_rank, rank, rot, spec.rot_dims,
+                       eps, spec.pairing)
+        q = linear(proj[:, :spec.q_rank], w["uq"])
+        c0 = spec.q_rank
+    else:
+        c0 = aligned_columns(H * (dim + rot), 0)[1]
+        latent_prepare(proj[:, c0:], pool, b.kv_rows, cos_sin, None, w["kv_norm"], 0, rank, rot, spec.rot_dims, eps,
+                       spec.pairing)
+        q = proj[:, :H * (dim + rot)]
     D = rank + rot
     qa = torch.empty((b.tokens, H * D), dtype=q.dtype, device=q.device)
     head_linear(qa, D, q, dim + rot, w["uk_t"])
@@ -264,7 +290,7 @@ def latent_attention_mixer(li: int, spec: LatentAttentionSpec, w: dict[str, torc
         sink_attention(lat, qa, pool, ctx.table, b.seq_start, b.seq_ctx, b.seq_slot, b.single_list, b.num_singles, 1,
                        None, *common, num_splits=splits, split_keys=per, window=spec.window, v_col0=0)
     out = torch.empty((b.tokens, H * spec.v_head_dim), dtype=q.dtype, device=q.device)
-    gate = proj[:, spec.q_rank + rank + rot:] if spec.out_gate else None
+    gate = proj[:, c0 + rank + rot:] if spec.out_gate else None
     head_linear(out, spec.v_head_dim, lat, rank, w["uv"], gate, spec.element_gate)
     return linear(out, w["o"])
 
@@ -489,7 +515,7 @@ def mlstm_mixer(li: int, spec: MlstmSpec, w: dict[str, torch.Tensor], x: torch.T
     return linear(head_norm_gate(y, w["norm"], H, eps, proj[:, g0:g0 + H * V], "sigmoid"), w["o"])
 
 
-def spec_magnitude(spec: BlockAttentionSpec) -> float:
+def spec_magnitude(spec: BlockAttentionSpec | LatentAttentionSpec) -> float:
     return rotary_frequencies(spec.rot_dims, spec.rot_base, spec.rot_factor, spec.rot_original, spec.rot_fast,
                               spec.rot_slow)[1]
 
@@ -505,10 +531,12 @@ def _activate(kind: str, x: torch.Tensor) -> torch.Tensor:
 
 
 def dense_feed_forward(spec: DenseMlpSpec, w: dict[str, torch.Tensor], x: torch.Tensor, reduce: bool = True) -> torch.Tensor:
-    if spec.gated:                                   # [gate | up] is one product; silu(gate) * up one kernel
+    if spec.gated:                                   # [gate | up] is one product; act(gate) * up one kernel
+        gu = linear(x, w["gate_up"])
+        if spec.activation == "gelu_tanh":
+            return linear(swiglu_scaled(gu[:, :spec.ff], gu[:, spec.ff:2 * spec.ff], form="gelu_tanh"), w["down"])
         if spec.activation != "silu":
             raise ValueError(f"unknown gated feed-forward activation {spec.activation!r}")
-        gu = linear(x, w["gate_up"])
         return linear(swiglu_forward(gu[:, :spec.ff], gu[:, spec.ff:]), w["down"])
     return linear(_activate(spec.activation, linear(x, w["up"])), w["down"])
 
@@ -516,10 +544,12 @@ def dense_feed_forward(spec: DenseMlpSpec, w: dict[str, torch.Tensor], x: torch.
 @dataclass
 class ExpertTerms:
     """A feed-forward's output as the rows its consumer sums: the chosen experts' weighted outputs ``[tokens, top, n]`` and
-    the shared expert's ``[tokens, n]``."""
+    the shared expert's ``[tokens, n]``; ``routed`` = (ids, weights, experts, input): a consumer of a design with identity
+    experts forms their terms itself, ``terms`` holds no rows for ids from ``experts`` on."""
 
     terms: torch.Tensor
     addend: torch.Tensor | None
+    routed: tuple[torch.Tensor, torch.Tensor, int, torch.Tensor] | None = None
 
 
 def moe_feed_forward(spec: MoeMlpSpec, w: dict[str, torch.Tensor], x: torch.Tensor,
@@ -528,7 +558,10 @@ def moe_feed_forward(spec: MoeMlpSpec, w: dict[str, torch.Tensor], x: torch.Tens
     the routed experts as two grouped products; the shared expert's output joins the weighted sum in its kernel
     (``reduce=False``: the terms are handed out for the consumer to sum)."""
     weights, ids = route_sigmoid_groups(x, w["router"], w.get("correction"), spec.top, spec.groups, spec.keep,
-                                        renormalize=spec.renormalize, scores=spec.scores, scale=spec.scale)
+                                        renormalize=spec.renormalize, scores=spec.scores, scale=spec.scale,
+                                        group_score=spec.group_score)
+    if spec.identity and reduce:
+        raise ValueError("identity experts: the consumer sums the terms")
     shared = None
     if spec.activation == "clamped":
         # the unit is formed in the grouped product's epilogue (gate and up rows interleaved); the shared expert's
@@ -536,11 +569,12 @@ def moe_feed_forward(spec: MoeMlpSpec, w: dict[str, torch.Tensor], x: torch.Tens
         if spec.shared_ff:
             f = spec.shared_ff
             gu = linear(x, w["shared_gate_up"])
-            shared = linear(swiglu_scaled(gu[:, :f], gu[:, f:2 * f], form="clamped", limit=spec.shared_limit,
+            z = gu[:, 2 * f:2 * f + 1] if spec.shared_gate else None     # the factor passes through the down product
+            shared = linear(swiglu_scaled(gu[:, :f], gu[:, f:2 * f], None, z, form="clamped", limit=spec.shared_limit,
                                           alpha=spec.alpha), w["shared_down"])
         out = grouped_experts(x, w["gate_up"], w["down"], weights, ids, addend=shared if reduce else None,
                               activation="clamped", gated=True, limit=spec.limit, alpha=spec.alpha, reduce=reduce)
-        return out if reduce else ExpertTerms(out, shared)
+        return out if reduce else ExpertTerms(out, shared, (ids, weights, spec.experts, x))
     if not reduce:
         raise ValueError("only the clamped experts hand out their terms")
     if spec.gated:
@@ -579,6 +613,8 @@ class LayeredDecoder:
         design soft-caps its logits)."""
         cfg, eps, off, kind = self.cfg, self.cfg.rms_norm_eps, self.norm_offset, self.cfg.norm_kind
         ctx = StepContext(batch, kv_buffer, table, states)
+        if kind == "tanh":
+            return self._forward_tanh_norm(tokens, ctx, want_rows)
         if cfg.streams:
             return self._forward_streams(tokens, ctx, want_rows)
         if cfg.single_norm:
@@ -692,6 +728,52 @@ class LayeredDecoder:
                 self.layer_trace.append(x.sum(1))
         if want_rows is not None and want_rows.numel() == 0:
             return torch.empty((0, cfg.vocab_size), dtype=torch.float32, device=tokens.device)
+        return self._logits(h)
+
+    def _forward_tanh_norm(self, tokens: torch.Tensor, ctx: StepContext, want_rows: torch.Tensor | None) -> torch.Tensor:
+        """``x <- x + sublayer(norm(x))`` with element-wise norms.  Between two sublayers ONE kernel adds the finished
+        sublayer to the fp32 residual (summing its expert terms), adds what the loop adds where a pass starts, and hands
+        out the next sublayer's input; the last one reads the wanted rows only, through the output norm."""
+        cfg, w = self.cfg, self.w
+        if not cfg.layers:
+            raise ValueError("tanh-norm designs have at least one layer")
+        subs = [(li, sub) for li, spec in enumerate(cfg.layers) for sub in range(1 if spec.mlp is None else 2)]
+        embedding = (tokens, w.embed, cfg.embed_scale)
+        resid = torch.empty((tokens.numel(), cfg.hidden_size), dtype=torch.float32, device=tokens.device)
+
+        def reads(at: int) -> dict:
+            """What sublayer ``at`` (past the end: the output) reads through and what comes into the residual before it."""
+            if at == len(subs):
+                return dict(norm=tuple(w.final_sub[n] for n in ("norm", "norm_b", "alpha")))
+            li, sub = subs[at]
+            out = dict(norm=tuple(w.layers[li].subs[sub][n] for n in ("norm", "norm_b", "alpha")))
+            t = cfg.layers[li].loop_pass if sub == 0 else None
+            if t is not None:
+                out.update(step=w.loop_step[t], embedding=embedding if t > 0 else None)
+            return out
+
+        h = tanh_norm_stream(resid, **{**reads(0), "embedding": embedding}, first=True)
+        for at, (li, sub) in enumerate(subs):
+            spec, lw = cfg.layers[li], w.layers[li]
+            if sub == 0:
+                y = MIXERS[spec.kind](li, spec.mixer, lw.mix, h, ctx, cfg.rms_norm_eps)
+            elif isinstance(spec.mlp, MoeMlpSpec):
+                y = FEED_FORWARDS[spec.mlp.kind](spec.mlp, lw.mlp, h, reduce=False)
+            else:
+                y = FEED_FORWARDS[spec.mlp.kind](spec.mlp, lw.mlp, h)
+            result = dict(y=y.terms, addend=y.addend, routed=y.routed) if isinstance(y, ExpertTerms) else dict(y=y)
+            last = at + 1 == len(subs)
+            if self.layer_trace is not None:                     # the residual before anything else joins
+                tanh_norm_stream(resid, **result)
+                result = {}
+                if last or subs[at + 1][0] != li:
+                    self.layer_trace.append(resid.clone())
+            if not last:
+                h = tanh_norm_stream(resid, **result, **reads(at + 1))
+            elif want_rows is None or want_rows.numel():
+                h = tanh_norm_stream(resid, **result, **reads(at + 1), rows=want_rows)
+        if want_rows is not None and want_rows.numel() == 0:
+            return torch.empty((0, cfg.vocab_size), dtype=self.dtype, device=tokens.device)
         return self._logits(h)
 
     def _forward_parallel(self, tokens: torch.Tensor, ctx: StepContext, want_rows: torch.Tensor | None) -> torch.Tensor:
@@ -1517,3 +1599,205 @@ _TORUTAR_SOURCES = ("gemm_dense", "gemm_simt", "gemm_rows_mma", "residual_stream
                     "elementwise")
 register(Architecture("Torutar", parse_torutar_config, map_torutar_weights, LayeredDecoder, ragged_steps=True,
                       sources=_TORUTAR_SOURCES))
+
+
+# --------------------------------------------------------------------------------------------- Povilorn plumbing #
+def _povilorn_mixer(kind: str, m: dict):
+    if kind == "attention":
+        qt = m.get("q_temp") or {}
+        return kind, SinkAttentionSpec(heads=int(m["heads"]), kv_heads=int(m.get("kv_heads", m["heads"])),
+                                       head_dim=int(m["dim"]), v_head_dim=int(m.get("vdim", m["dim"])),
+                                       scale=float(m["scale"]), gain_coef=float(qt.get("coef", 0.0)),
+                                       gain_every=float(qt.get("every", 0.0)), keys_as_values=True, element_gate=True)
+    if kind == "latent_attention":
+        rot_dim = int(m.get("rot_dim", 0))
+        rot = m.get("rot") or {}
+        sc = rot.get("scaling") or {}
+        return kind, LatentAttentionSpec(
+            heads=int(m["heads"]), head_dim=int(m["dim"]), rot_dim=rot_dim, v_head_dim=int(m.get("vdim", m["dim"])),
+            q_rank=0, kv_rank=int(m["kv_rank"]), scale=float(m["scale"]), rot_dims=int(rot.get("dims", rot_dim)),
+            rot_base=float(rot.get("base", 10000.0)), out_gate=False, pairing="neighbours",
+            rot_factor=float(sc.get("factor", 1.0)), rot_original=float(sc.get("original", 0.0)),
+            rot_fast=float(sc.get("fast", 0.0)), rot_slow=float(sc.get("slow", 0.0)))
+    raise ValueError(f"unknown layer type {kind!r}")
+
+
+def _povilorn_mlp(mlp: dict | None) -> DenseMlpSpec | MoeMlpSpec | None:
+    if mlp is None:
+        return None
+    kind = mlp.get("kind", "dense")
+    if kind == "dense":
+        return DenseMlpSpec(ff=int(mlp["ff"]), activation="gelu_tanh", gated=True)
+    if kind != "moe":
+        raise ValueError(f"unknown feed-forward kind {kind!r}")
+    r, shared = mlp["router"], mlp.get("shared") or {}
+    groups = r.get("groups") or {}
+    return MoeMlpSpec(experts=int(r["experts"]), top=int(r["top"]), ff=int(mlp["expert"]["ff"]),
+                      groups=int(groups.get("count", 1)), keep=int(groups.get("keep", groups.get("count", 1))),
+                      shared_ff=int(shared.get("ff", 0)), activation="clamped", gated=True, shared_gate=bool(shared),
+                      scores="softmax", limit=float(mlp["expert"]["limit"]), shared_limit=float(shared.get("limit", 0.0)),
+                      identity=int(r.get("identity", 0)), group_score="max")
+
+
+def looped_order(count: int, loop: dict | None) -> list[tuple[int, int | None]]:
+    """The runs of ``count`` layers of which ``start .. stop - 1`` run ``times`` times in a row: (layer, pass number on the
+    first layer of a pass, else None)."""
+    if not loop:
+        return [(i, None) for i in range(count)]
+    start, stop, times = int(loop["start"]), int(loop["stop"]), int(loop["times"])
+    if not 0 <= start < stop <= count or times < 1:
+        raise ValueError(f"a loop over layers {start} .. {stop - 1} of {count}, {times} times")
+    body = [(i, t if i == start else None) for t in range(times) for i in range(start, stop)]
+    return [(i, None) for i in range(start)] + body + [(i, None) for i in range(stop, count)]
+
+
+def parse_povilorn_config(raw: dict) -> LayeredConfig:
+    stored = []
+    for entry in raw["layers"]:
+        key, mixer = _povilorn_mixer(entry["type"], entry["mixer"])
+        stored.append(LayerSpec(key, mixer, _povilorn_mlp(entry.get("mlp"))))
+    layers, owner = [], {}
+    for i, t in looped_order(len(stored), raw.get("loop")):
+        s = stored[i]
+        layers.append(LayerSpec(s.kind, s.mixer, s.mlp, weights_of=owner.get(i), source=i, loop_pass=t))
+        owner.setdefault(i, len(layers) - 1)
+    return LayeredConfig(name=raw.get("architecture", "Povilorn"), hidden_size=int(raw["width"]),
+                         vocab_size=int(raw["vocab"]), max_seq_len=0, rms_norm_eps=float(raw["norm"]["eps"]),
+                         layers=tuple(layers), norm_kind="tanh", norm_weight_offset=0.0, learned_positions=False,
+                         embed_scale=float((raw.get("embedding") or {}).get("scale", 1.0)),
+                         loop_passes=int(raw["loop"]["times"]) if raw.get("loop") else 0)
+
+
+def map_povilorn_weights(cfg: LayeredConfig, tensors: dict[str, torch.Tensor], device: str,
+                         dtype: torch.dtype) -> LayeredWeights:
+    """Checkpoint names -> the decoder's weights.  Every mixer's input projections are row-concatenated into one GEMM
+    weight (parts that a kernel reads with 16-byte accesses start on a multiple of 8 rows), with one bias vector where some
+    part has a bias; the query and key norm weights of a layer whose keys are its values are multiplied per query entry
+    (fp32); the latent key up-projection is stored transposed per head; experts are stacked with each expert's gate and up
+    rows interleaved, the shared expert's token-gate row rides at the end of its [gate | up] weight.  Every run of a
+    looped layer gets the very object of its first run."""
+
+    def get(name: str, dt: torch.dtype = dtype) -> torch.Tensor:
+        if name not in tensors:
+            raise KeyError(f"checkpoint has no tensor {name!r}")
+        return tensors[name].to(device=device, dtype=dt).contiguous()
+
+    def norm(name: str) -> dict[str, torch.Tensor]:
+        return {"norm": get(name), "norm_b": get(name + ".b"), "alpha": get(name + ".alpha").reshape(1)}
+
+    final = norm("final.norm")
+    out = LayeredWeights(embed=get("embed"), pos=None, final_norm=final["norm"], head=get("head"), final_sub=final,
+                         loop_step=get("loop.step") if cfg.loop_passes else None)
+    freq_cache: dict[tuple, torch.Tensor] = {}
+    built: list[LayeredLayerWeights] = []
+    for run in cfg.layers:
+        if run.weights_of is not None:
+            built.append(built[run.weights_of])
+            continue
+        i, m = run.source, run.mixer
+        p = f"l{i}.mix."
+        if isinstance(m, SinkAttentionSpec):
+            per = m.heads // m.kv_heads
+            wk = get(p + "k.norm", torch.float32).view(m.kv_heads, 1, m.head_dim).expand(-1, per, -1).reshape(-1)
+            bias = torch.cat([get(p + "q.b"), get(p + "k.b")])
+            mix = {"qkv": _stack_aligned([torch.cat([get(p + "q"), get(p + "k")], dim=0), get(p + "g")]),
+                   "query_weight": (get(p + "q.norm", torch.float32) * wk).contiguous(), "o": get(p + "o")}
+            mix["qkv_b"] = torch.zeros(mix["qkv"].shape[0], dtype=dtype, device=device)
+            mix["qkv_b"][:bias.numel()] = bias
+        else:
+            uk = get(p + "uk").view(m.heads, m.head_dim, m.kv_rank)
+            mix = {"down": _stack_aligned([get(p + "q"), get(p + "dkv")]), "kv_norm": get(p + "dkv.norm"),
+                   "uk_t": uk.transpose(1, 2).contiguous(),
+                   "uv": get(p + "uv").view(m.heads, m.v_head_dim, m.kv_rank).contiguous(), "o": get(p + "o")}
+            key = (m.rot_dims, m.rot_base, m.rot_factor, m.rot_original, m.rot_fast, m.rot_slow)
+            if m.rot_dims:
+                if key not in freq_cache:
+                    freq_cache[key] = torch.tensor(rotary_frequencies(*key)[0], dtype=torch.float64).to(device=device)
+                mix["freqs"] = freq_cache[key]
+        lw = LayeredLayerWeights(norm1=None, mix=mix, subs=[norm(f"l{i}.norm1")])
+        q = f"l{i}.mlp."
+        if run.mlp is not None:
+            lw.subs.append(norm(f"l{i}.norm2"))
+        if isinstance(run.mlp, DenseMlpSpec):
+            lw.mlp = {"gate_up": torch.cat([get(q + "gate"), get(q + "up")], dim=0).contiguous(), "down": get(q + "down")}
+        elif isinstance(run.mlp, MoeMlpSpec):
+            e = range(run.mlp.experts)
+            lw.mlp = {"router": get(q + "router"),
+                      "gate_up": torch.stack([torch.stack([get(f"{q}e{j}.gate"), get(f"{q}e{j}.up")], dim=1).flatten(0, 1)
+                                              for j in e]).contiguous(),
+                      "down": torch.stack([get(f"{q}e{j}.down") for j in e]).contiguous()}
+            if q + "correction" in tensors:
+                lw.mlp["correction"] = get(q + "correction")
+            if run.mlp.shared_ff:
+                lw.mlp["shared_gate_up"] = _pad_rows(torch.cat([get(q + "shared.gate"), get(q + "shared.up"),
+                                                                get(q + "shared.sg").reshape(1, -1)], dim=0), 8).contiguous()
+                lw.mlp["shared_down"] = get(q + "shared.down")
+        built.append(lw)
+    out.layers = built
+    return out
+
+
+def povilorn_tensor_shapes(cfg: LayeredConfig) -> dict[str, tuple[int, ...]]:
+    """Checkpoint tensor names and shapes of a configuration (random initialisation, shape checks)."""
+    w = cfg.hidden_size
+
+    def norm(name: str) -> dict[str, tuple[int, ...]]:
+        return {name: (w,), name + ".b": (w,), name + ".alpha": ()}
+
+    shapes: dict[str, tuple[int, ...]] = {"embed": (cfg.vocab_size, w)}
+    if cfg.loop_passes:
+        shapes["loop.step"] = (cfg.loop_passes, w)
+    for run in cfg.layers:
+        if run.weights_of is not None:
+            continue
+        p, m = f"l{run.source}.mix.", run.mixer
+        shapes.update(norm(f"l{run.source}.norm1"))
+        if isinstance(m, SinkAttentionSpec):
+            nq, nk = m.heads * m.head_dim, m.kv_heads * m.head_dim
+            shapes.update({p + "q": (nq, w), p + "q.b": (nq,), p + "k": (nk, w), p + "k.b": (nk,), p + "q.norm": (nq,),
+                           p + "k.norm": (nk,), p + "g": (nq, w), p + "o": (w, nq)})
+        else:
+            shapes.update({p + "q": (m.heads * (m.head_dim + m.rot_dim), w), p + "dkv": (m.kv_rank + m.rot_dim, w),
+                           p + "dkv.norm": (m.kv_rank,), p + "uk": (m.heads * m.head_dim, m.kv_rank),
+                           p + "uv": (m.heads * m.v_head_dim, m.kv_rank), p + "o": (w, m.heads * m.v_head_dim)})
+        q, f = f"l{run.source}.mlp.", run.mlp
+        if f is None:
+            continue
+        shapes.update(norm(f"l{run.source}.norm2"))
+        if isinstance(f, DenseMlpSpec):
+            shapes.update({q + "gate": (f.ff, w), q + "up": (f.ff, w), q + "down": (w, f.ff)})
+            continue
+        for e in [*(f"e{j}" for j in range(f.experts)), *(["shared"] if f.shared_ff else [])]:
+            ff = f.shared_ff if e == "shared" else f.ff
+            shapes.update({f"{q}{e}.gate": (ff, w), f"{q}{e}.up": (ff, w), f"{q}{e}.down": (w, ff)})
+        shapes.update({q + "router": (f.choices, w), q + "correction": (f.choices,)})
+        if f.shared_ff:
+            shapes[q + "shared.sg"] = (1, w)
+    shapes.update({**norm("final.norm"), "head": (cfg.vocab_size, w)})
+    return shapes
+
+
+def random_povilorn_tensors(cfg: LayeredConfig, seed: int = 0) -> dict[str, torch.Tensor]:
+    """Seeded random bf16 tensors with checkpoint names (benchmarks and tests; no trained checkpoints exist offline)."""
+    g = torch.Generator().manual_seed(seed)
+    out = {}
+    for name, shape in povilorn_tensor_shapes(cfg).items():
+        leaf = name.rsplit(".", 1)[-1]
+        if leaf == "alpha":
+            t = torch.tensor(0.5)
+        elif name == "loop.step" or leaf == "b":
+            t = 0.3 * torch.randn(shape, generator=g)
+        elif len(shape) == 2:
+            t = torch.randn(shape, generator=g) / (shape[1] ** 0.5)
+        elif leaf == "correction":
+            t = 0.02 * torch.randn(shape, generator=g)
+        else:                                                 # norm weights
+            t = 1.0 + 0.1 * torch.randn(shape, generator=g)
+        out[name] = t.to(torch.bfloat16)
+    return out
+
+
+_POVILORN_SOURCES = ("gemm_dense", "gemm_simt", "gemm_rows_mma", "gated_linear_attention", "tanh_norm_stream", "rotary_heads",
+                     "latent_attention", "attention_sink", "moe_routing", "elementwise")
+register(Architecture("Povilorn", parse_povilorn_config, map_povilorn_weights, LayeredDecoder, ragged_steps=True,
+                      sources=_POVILORN_SOURCES))

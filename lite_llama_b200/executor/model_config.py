@@ -116,7 +116,10 @@ class Mamba2Spec:
 class SinkAttentionSpec:
     """Position-free attention: whole-row q / k norms, a query gain that grows with the logarithm of the position
     (``1 + gain_coef * ln(floor((p + 1) / gain_every) + 1)``; ``gain_every == 0``: none), ``tanh`` soft cap
-    (0: none), a learned per-head sink in the softmax denominator, value mixing across the layers that ask for it."""
+    (0: none), a learned per-head sink in the softmax denominator, value mixing across the layers that ask for it.
+    ``keys_as_values``: there are no values of their own, the projected keys (before the key norm) are the values; a pool
+    row then holds each key once, as projected, and the key norm's statistic.  ``element_gate``: the joined heads are
+    multiplied by the logistic function of a projection of the mixer input before the output projection."""
 
     heads: int
     kv_heads: int
@@ -127,13 +130,18 @@ class SinkAttentionSpec:
     gain_coef: float = 0.0
     gain_every: float = 0.0
     v_mix: bool = False
+    keys_as_values: bool = False
+    element_gate: bool = False
 
     def validate(self) -> None:
-        if self.heads % self.kv_heads or self.v_head_dim > 256:
+        if self.heads % self.kv_heads or self.v_head_dim > 256 or \
+                (self.keys_as_values and (self.v_head_dim != self.head_dim or self.v_mix)):
             raise ValueError(f"unsupported attention geometry: {self}")
 
     @property
     def cache_row_width(self) -> int:                  # one token's pool row: all K heads, then all V heads
+        if self.keys_as_values:                        # all K heads, a 4-byte statistic; padded to 16-byte vectors
+            return -(-(self.kv_heads * self.head_dim + 3) // 8) * 8
         return self.kv_heads * (self.head_dim + self.v_head_dim)
 
 
@@ -142,7 +150,8 @@ class LatentAttentionSpec:
     """Attention through low-rank latents: queries ``h -> q_rank -> heads x (head_dim + rot_dim)``; keys / values
     ``h -> kv_rank`` (the cached latent) ``-> heads x head_dim`` keys and ``heads x v_head_dim`` values, plus one
     ``rot_dim``-wide rotated key part shared by all heads (cached beside the latent).  Rotary positions act on the
-    first ``rot_dims`` entries of the rotated parts (rotate-half pairing, base ``rot_base``).  ``window`` > 0: a token
+    first ``rot_dims`` entries of the rotated parts (``pairing``, base ``rot_base``, with ``rot_factor`` > 1 the frequency
+    interpolation of ``kernels.rotary_frequencies``).  ``q_rank = 0``: queries come straight from ``h``.  ``window`` > 0: a token
     sees itself and the ``window - 1`` tokens before it.  ``out_gate``: a per-head sigmoid gate on the head outputs."""
 
     heads: int
@@ -158,9 +167,13 @@ class LatentAttentionSpec:
     out_gate: bool = True
     element_gate: bool = False                         # out_gate has one number per output element instead of per head
     pairing: str = "halves"                            # rotary pairs: i, i + rot_dims / 2; "neighbours": 2i, 2i + 1
+    rot_factor: float = 1.0
+    rot_original: float = 0.0
+    rot_fast: float = 0.0
+    rot_slow: float = 0.0
 
     def validate(self) -> None:
-        if min(self.heads, self.head_dim, self.v_head_dim, self.q_rank, self.kv_rank) < 1 or self.rot_dim < 0 or \
+        if min(self.heads, self.head_dim, self.v_head_dim, self.kv_rank) < 1 or min(self.rot_dim, self.q_rank) < 0 or \
                 self.rot_dims % 2 or not 0 <= self.rot_dims <= self.rot_dim or self.window < 0 or self.kv_rank > 256 or \
                 self.pairing not in ("neighbours", "halves"):
             raise ValueError(f"unsupported latent attention geometry: {self}")
@@ -466,7 +479,7 @@ class MlstmSpec:
 @dataclass(frozen=True)
 class DenseMlpSpec:
     ff: int
-    activation: str = "relu2"                          # "relu2" | "gelu" | "gelu_tanh"; gated: "silu"
+    activation: str = "relu2"                          # "relu2" | "gelu" | "gelu_tanh"; gated: "silu" | "gelu_tanh"
     kind: str = "dense"                                # key of executor.layered_decoder.FEED_FORWARDS
     gated: bool = False                                # W_down (act(W_gate h) * (W_up h)) instead of W_down act(W_up h)
 
@@ -481,7 +494,9 @@ class MoeMlpSpec:
     weighted.  ``shared_gate``: the shared expert's output is scaled by one logistic number per token.
     ``scores="softmax"``: the scores are the softmax over all experts.  ``scale`` multiplies the weights.
     ``activation="clamped"`` (gated): ``g' sigmoid(alpha g') (u' + 1)`` with ``g' = min(g, limit)`` and
-    ``u' = clamp(u, -limit, limit)``; the shared expert's bound is ``shared_limit``."""
+    ``u' = clamp(u, -limit, limit)``; the shared expert's bound is ``shared_limit``.  ``identity``: that many router rows
+    after the experts' are identity experts, whose output is their input; they take part in scores, groups and choice.
+    ``group_score="max"``: a group competes with its best choice score alone."""
 
     experts: int
     top: int
@@ -500,10 +515,17 @@ class MoeMlpSpec:
     limit: float = 0.0
     shared_limit: float = 0.0
     alpha: float = 1.702
+    identity: int = 0
+    group_score: str = "top2"
+
+    @property
+    def choices(self) -> int:                          # what the router chooses among
+        return self.experts + self.identity
 
     def validate(self) -> None:
-        if self.experts < 1 or not 1 <= self.top <= self.experts or self.groups < 1 or self.experts % self.groups or \
-                not 1 <= self.keep <= self.groups or self.keep * (self.experts // self.groups) < self.top:
+        if self.experts < 1 or self.identity < 0 or not 1 <= self.top <= self.choices or self.groups < 1 or \
+                self.choices % self.groups or not 1 <= self.keep <= self.groups or \
+                self.keep * (self.choices // self.groups) < self.top or self.group_score not in ("top2", "max"):
             raise ValueError(f"unsupported expert routing: {self}")
 
 
@@ -513,6 +535,8 @@ class LayerSpec:
     mixer: "Mamba2Spec | SinkAttentionSpec | LatentAttentionSpec | MinGruSpec | RgLruSpec | SideBySideSpec | WindowAttentionSpec | MlstmSpec"
     mlp: DenseMlpSpec | MoeMlpSpec | None = None
     weights_of: int | None = None                      # the layer whose tensors this one uses (cache / state are its own)
+    source: int | None = None                          # looped designs: the checkpoint layer this run of it belongs to
+    loop_pass: int | None = None                       # set on the first layer of a pass of the loop: the pass's number
 
 
 @dataclass(frozen=True)
@@ -523,7 +547,9 @@ class LayeredConfig:
     max_seq_len: int                                   # learned position table length; 0 = bounded by the KV pool only
     rms_norm_eps: float
     layers: tuple[LayerSpec, ...] = ()
-    norm_kind: str = "rms"                             # "rms" | "layer" (layer norm with a weight, no bias)
+    # "rms" | "layer" (layer norm with a weight, no bias) | "tanh" (element-wise: tanh(alpha x) * w + b; x <- x +
+    # sublayer(norm(x)) without output norms)
+    norm_kind: str = "rms"
     pre_norm: bool = False                             # sublayers read norm(x) (with norms on their outputs as well)
     layer_scale: bool = False                          # per-channel scale on each sublayer's normed output
     norm_weight_offset: float = 1.0                    # 1: norm weights stored around zero; 0: plain weights
@@ -548,6 +574,10 @@ class LayeredConfig:
     streams: int = 0
     input_conv: int = 0
     sublayer_gate: bool = False
+    # a looped design runs some of its layers several times: ``layers`` lists the RUNS in order (later passes name the first
+    # one in ``weights_of``, every run has a cache of its own); where a pass starts (``loop_pass``) the embedding output
+    # (but for the first pass) and the pass's own vector are added to the residual.  loop_passes: how many vectors there are
+    loop_passes: int = 0
 
     @property
     def num_layers(self) -> int:
@@ -568,6 +598,8 @@ class LayeredConfig:
     def validate(self) -> None:
         for i, l in enumerate(self.layers):
             l.mixer.validate()
+            if l.loop_pass is not None and not (0 <= l.loop_pass < self.loop_passes and self.norm_kind == "tanh"):
+                raise ValueError(f"layer {i} starts pass {l.loop_pass} of {self.loop_passes}")
             if isinstance(l.mlp, MoeMlpSpec):
                 l.mlp.validate()
             if l.weights_of is not None:

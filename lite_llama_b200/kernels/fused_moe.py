@@ -10,6 +10,7 @@ from ._common import check, dtype_code, float_code, index_width, lib, ptr, requi
 
 _KIND_F16, _KIND_FP8, _KIND_INT8 = 0, 1, 2
 SCORES = {"sigmoid": 0, "softmax": 1}
+GROUP_SCORES = {"top2": 0, "max": 1}
 
 
 @torch.no_grad()
@@ -171,11 +172,11 @@ def route_topk(router_logits: torch.Tensor, top_k: int, renormalize: bool = True
 @torch.no_grad()
 def route_sigmoid_groups(x: torch.Tensor, router_w: torch.Tensor, bias: torch.Tensor | None, top_k: int,
                          groups: int = 1, keep: int = 1, renormalize: bool = True, scores: str = "sigmoid",
-                         scale: float = 1.0):
+                         scale: float = 1.0, group_score: str = "top2"):
     """Sigmoid router with a selection bias and group-limited choice (router product with fp32 results + one selection
     launch; a single launch for shapes no GEMM takes):
     ``s = sigmoid(router_w @ x)`` (``scores="softmax"``: the softmax over all experts) in fp32; experts compete with ``s + bias``; they form ``groups`` runs of neighbours,
-    a group scores the sum of its two best, only the ``keep`` best groups are eligible; the ``top_k`` winners' weights
+    a group scores the sum of its two best (``group_score="max"``: its best), only the ``keep`` best groups are eligible; the ``top_k`` winners' weights
     are their ``s`` over the winners' sum (``renormalize=False``: their ``s`` as they are), times ``scale``.  Returns ``(weights fp32 [T, k], ids int32 [T, k])``.  The reference's
     router is a softmax over all experts (lite_llama/models/qwen3_moe.py:94-100, ``route_topk``)."""
     require_cuda(x, router_w, bias)
@@ -202,6 +203,7 @@ def route_sigmoid_groups(x: torch.Tensor, router_w: torch.Tensor, bias: torch.Te
                                       code, stream_handle()))
     check(L.b2l_moe_route_sigmoid_groups(w.data_ptr(), ids.data_ptr(), x.data_ptr(), x.stride(0), router_w.data_ptr(),
                                          ptr(bias), ptr(logits), tokens, e, k, int(top_k), int(groups), int(keep),
+                                         GROUP_SCORES[group_score],
                                          1 if renormalize else 0, SCORES[scores], float(scale), code, stream_handle()))
     return w, ids
 
@@ -229,7 +231,8 @@ def grouped_experts(x: torch.Tensor, w_up: torch.Tensor, w_down: torch.Tensor, w
     ``activation="clamped"`` (gated): ``w_up`` interleaves every expert's rows (2i: gate i, 2i + 1: up i) and the unit
     ``g' sigmoid(alpha g') (u' + 1)``, ``g' = min(g, limit)``, ``u' = clamp(u, -limit, limit)`` is formed from the fp32
     sums in the first product's epilogue, so the two halves are never stored.  ``reduce=False``: the weighted outputs
-    of a token's experts are returned as ``[tokens, top_k, h]`` for a consumer that sums them itself.  The fp16 / fp8 gated experts
+    of a token's experts are returned as ``[tokens, top_k, h]`` for a consumer that sums them itself; ids from
+    ``len(w_up)`` on (experts without weights) get no rows there, what those places hold is undefined.  The fp16 / fp8 gated experts
     of the reference's family are ``fused_moe``."""
     require_cuda(x, w_up, w_down, weights, ids, addend)
     if (activation, gated) not in (("gelu", False), ("silu", True), ("clamped", True)) or \

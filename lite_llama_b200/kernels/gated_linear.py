@@ -7,7 +7,7 @@ import torch
 
 from ._common import check, counters, float_code, lib, ptr, require_cuda, stream_handle
 
-GATED_UNITS = {"silu": 0, "clamped": 1}
+GATED_UNITS = {"silu": 0, "clamped": 1, "gelu_tanh": 2}
 GATED_LINEAR_MODES = {"forget_gate": 0, "delta_rule": 1}
 
 
@@ -131,7 +131,8 @@ def swiglu_scaled(gate: torch.Tensor, up: torch.Tensor, in_scale: torch.Tensor |
     """``silu(s * gate) * (s * up) * sigmoid(z)`` with one fp32 factor ``s = in_scale[r]`` and one logit
     ``z = out_logit[r, 0]`` per row (both optional).  A factor on a gated unit's INPUT passes through its two linear
     maps, so it is applied here, between the products and the activation.  ``form="clamped"``: the unit is
-    ``g' sigmoid(alpha g') (u' + 1)`` with ``g' = min(g, limit)``, ``u' = clamp(u, -limit, limit)`` instead."""
+    ``g' sigmoid(alpha g') (u' + 1)`` with ``g' = min(g, limit)``, ``u' = clamp(u, -limit, limit)`` instead;
+    ``form="gelu_tanh"``: ``gelu(g) * u`` with the tanh form of GELU."""
     require_cuda(gate, up, in_scale, out_logit)
     rows, n = gate.shape
     if up.shape != gate.shape or gate.stride(-1) != 1 or up.stride(-1) != 1 or up.dtype != gate.dtype or \

@@ -26,16 +26,16 @@ def rope_table(positions: torch.Tensor, rot_dims: int, rot_base: float) -> torch
 
 @torch.no_grad()
 def latent_prepare(proj: torch.Tensor, pool: torch.Tensor, kv_rows: torch.Tensor, cos_sin: torch.Tensor | None,
-                   q_norm: torch.Tensor, kv_norm: torch.Tensor, q_rank: int, kv_rank: int, rot_dim: int,
+                   q_norm: torch.Tensor | None, kv_norm: torch.Tensor, q_rank: int, kv_rank: int, rot_dim: int,
                    rot_dims: int, eps: float, pairing: str = "halves") -> None:
     """Per token of the fused down-projection ``proj [T, >= q_rank + kv_rank + rot_dim]``: RMS norm of the query latent
-    in place, RMS norm of the key/value latent and the rotation (``rope_table`` rows) of the shared key part into pool
+    in place (``q_rank = 0``: there is none), RMS norm of the key/value latent and the rotation (``rope_table`` rows) of the shared key part into pool
     row ``kv_rows[t]``."""
     require_cuda(proj, pool, kv_rows, cos_sin, q_norm, kv_norm)
     if proj.stride(-1) != 1 or pool.stride(-1) != 1 or pool.shape[1] < kv_rank + rot_dim:
         raise ValueError("latent_prepare: bad layout")
     check(lib().b2l_latent_prepare(proj.data_ptr(), proj.stride(0), pool.data_ptr(), pool.stride(0), kv_rows.data_ptr(),
-                                   ptr(cos_sin), q_norm.data_ptr(), kv_norm.data_ptr(), proj.shape[0], q_rank,
+                                   ptr(cos_sin), ptr(q_norm), kv_norm.data_ptr(), proj.shape[0], q_rank,
                                    kv_rank, rot_dim, rot_dims, PAIRINGS[pairing], float(eps), float_code(proj, "proj"),
                                    stream_handle()))
 
