@@ -1,9 +1,9 @@
-"""``bench.py --design gufotar | pesivik | tisosun | gofezen | torutar``: prefill and decode throughput of a layer-list design at a few sizes that resemble
+"""``bench.py --design gufotar | pesivik | tisosun | gofezen | torutar | povilorn``: prefill and decode throughput of a layer-list design at a few sizes that resemble
 a real model's layers (random weights, synthetic ids), beside the closest existing model of the framework (the
 uniform rotary decoder: same width, layer count, attention geometry and feed-forward width; for Tisosun the Gufotar
 layer-list model, the other design with recurrent layers beside attention layers; for Gofezen the Tisosun model, the
 other design of parallel blocks; for Torutar the Gofezen model, the other design of window attention, memories and gated
-routed experts), plus every kernel of the
+routed experts; for Povilorn the Pesivik model, the other design of latent attention and experts in groups), plus every kernel of the
 new path timed alone against its like kernel with the fraction of the measured roofline each reaches.
 
 Timing: CUDA events on the launching stream, >= 3 warm-up runs, a 256 MiB write between timed runs (larger than the
@@ -1306,6 +1306,231 @@ def torutar_kernel_table(sz, batch, prompt, dev, dtype, flush, hbm_gbs, tflops) 
     return rows
 
 
+# ----------------------------------------------------------------------------------------------------- Povilorn #
+V_SIZES = {
+    # layers in turn: latent attention (l_dim + rot per head over a cached row of kv_rank + rot) with a dense feed-forward;
+    # attention whose values are its keys (heads x head_dim on kv_heads) with routed, identity and shared experts.  The first
+    # two layers run `times` times, `layers` counts the runs.  q_rank and window are the Pesivik geometry's own columns
+    "small": dict(width=1024, layers=4, times=2, heads=16, kv_heads=4, head_dim=64, every=256, l_dim=64, rot=32, kv_rank=128,
+                  dense=2048, experts=16, identity=8, top=4, groups=4, keep=2, e_ff=512, shared=1024, vocab=32000, q_rank=384),
+    "1b": dict(width=2048, layers=8, times=2, heads=16, kv_heads=4, head_dim=128, every=256, l_dim=128, rot=64, kv_rank=256,
+               dense=8192, experts=32, identity=16, top=4, groups=4, keep=2, e_ff=1024, shared=2048, vocab=32000, q_rank=768),
+    "8b": dict(width=4096, layers=8, times=2, heads=32, kv_heads=8, head_dim=128, every=256, l_dim=128, rot=64, kv_rank=256,
+               dense=14336, experts=64, identity=32, top=8, groups=8, keep=4, e_ff=1024, shared=2048, vocab=32000, q_rank=1536),
+}
+V_SCALING = {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}
+
+
+def povilorn_config(sz: dict) -> dict:
+    lat = {"type": "latent_attention",
+           "mixer": {"heads": sz["heads"], "dim": sz["l_dim"], "rot_dim": sz["rot"], "vdim": sz["l_dim"], "kv_rank": sz["kv_rank"],
+                     "scale": 1.0 / math.sqrt(sz["l_dim"] + sz["rot"]),
+                     "rot": {"dims": sz["rot"], "base": 10000.0, "scaling": V_SCALING}},
+           "mlp": {"kind": "dense", "ff": sz["dense"]}}
+    att = {"type": "attention",
+           "mixer": {"heads": sz["heads"], "kv_heads": sz["kv_heads"], "dim": sz["head_dim"], "vdim": sz["head_dim"],
+                     "scale": 1.0 / math.sqrt(sz["head_dim"]), "q_temp": {"coef": 0.1, "every": sz["every"]}},
+           "mlp": {"kind": "moe", "expert": {"ff": sz["e_ff"], "limit": 7.0}, "shared": {"ff": sz["shared"], "limit": 6.0},
+                   "router": {"experts": sz["experts"], "identity": sz["identity"], "top": sz["top"],
+                              "groups": {"count": sz["groups"], "keep": sz["keep"]}}}}
+    stored = sz["layers"] - 2 * (sz["times"] - 1)
+    return {"architecture": "Povilorn", "width": sz["width"], "vocab": sz["vocab"], "norm": {"eps": 1e-6},
+            "embedding": {"scale": 2.0}, "loop": {"start": 0, "stop": 2, "times": sz["times"]},
+            "layers": [(lat, att)[i % 2] for i in range(stored)]}
+
+
+def build_povilorn(sz, batch, max_positions, dev, dtype):
+    from lite_llama_b200.executor import ModelRunner
+    from lite_llama_b200.executor.layered_decoder import map_povilorn_weights, parse_povilorn_config, random_povilorn_tensors
+
+    conf = parse_povilorn_config(povilorn_config(sz))
+    conf.validate()
+    weights = map_povilorn_weights(conf, random_povilorn_tensors(conf, seed=0), dev, dtype)
+    return ModelRunner(conf, weights, batch * max_positions, device=dev, dtype=dtype, max_requests=batch)
+
+
+def povilorn_step_throughput(sz, batch, prompt, dev, dtype, flush) -> dict:
+    """tokens/s of a whole-prompt step and of a decode step: Povilorn beside the Pesivik model (the other design of latent
+    attention and routed experts in groups) of the same width, layer runs, heads, latent sizes, expert count and expert
+    width, without a window."""
+    like = dict(width=sz["width"], layers=sz["layers"], heads=sz["heads"], dim=sz["l_dim"], rot_dim=sz["rot"], vdim=sz["l_dim"],
+                q_rank=sz["q_rank"], kv_rank=sz["kv_rank"], window=0, experts=sz["experts"], top=sz["top"], groups=sz["groups"],
+                keep=sz["keep"], ff=sz["e_ff"], shared_ff=sz["shared"], vocab=sz["vocab"])
+    return _layered_steps((("povilorn", lambda m: build_povilorn(sz, batch, m, dev, dtype)),
+                           ("pesivik", lambda m: build_pesivik(like, batch, m, dev, dtype))), sz, batch, prompt, flush)
+
+
+def povilorn_kernel_table(sz, batch, prompt, dev, dtype, flush, hbm_gbs, tflops) -> list[dict]:
+    """Every kernel of the Povilorn path alone at the size's shapes beside its like kernel of the Pesivik path (plain
+    attention: of the Gufotar path), with the fraction of the measured roofline each reaches."""
+    import lite_llama_b200.kernels as K
+    from lite_llama_b200.executor.layered_decoder import split_plan
+
+    es = 2
+    W, H, G, D = sz["width"], sz["heads"], sz["kv_heads"], sz["head_dim"]
+    dim, rot, kr, qr = sz["l_dim"], sz["rot"], sz["kv_rank"], sz["q_rank"]
+    E, I, top, ff, sff, dff = sz["experts"], sz["identity"], sz["top"], sz["e_ff"], sz["shared"], sz["dense"]
+    T, ctx = batch * prompt, prompt
+    rows: list[dict] = []
+
+    def i32(v):
+        return torch.tensor(list(v), dtype=torch.int32, device=dev)
+
+    def rnd(*shape, dt=dtype, s=1.0):
+        return (torch.randn(*shape, device=dev) * s).to(dt)
+
+    def add(name, like, fn, nbytes=0, flops=0, like_fn=None, like_bytes=None, like_flops=None):
+        ms = timed(fn, flush)
+        row = {"kernel": name, "us": ms * 1e3}
+        if flops:
+            row.update(tflops=flops / ms / 1e9, frac=flops / ms / 1e9 / tflops, bound="tensor")
+        else:
+            row.update(gbs=nbytes / ms / 1e6, frac=nbytes / ms / 1e6 / hbm_gbs, bound="hbm")
+        if like_fn is not None:
+            lms = timed(like_fn, flush)
+            lf = like_flops if like_flops is not None else flops
+            lb = like_bytes if like_bytes is not None else nbytes
+            lfrac = lf / lms / 1e9 / tflops if flops else lb / lms / 1e6 / hbm_gbs
+            row.update(like=like, like_us=lms * 1e3, like_frac=lfrac,
+                       distance_ratio=(lfrac / row["frac"]) if row["frac"] else None)
+        rows.append(row)
+
+    p_start, p_ctx, p_slot = i32(range(0, T + 1, prompt)), i32([0] * batch), i32(range(batch))
+    d_start, d_ctx = i32(range(batch + 1)), i32([ctx] * batch)
+    # ---------------- the residual between two sublayers
+    nw, nb, alpha = rnd(W, s=0.1) + 1, rnd(W, s=0.1), rnd(1) + 1
+    wn, ls = rnd(W, s=0.1) + 1, rnd(W, s=0.1) + 0.5
+    emb, toks = rnd(sz["vocab"], W), torch.randint(0, sz["vocab"], (T,), dtype=torch.int32, device=dev)
+    step = rnd(W)
+    for name, n in (("prompts", T), ("decode", batch)):
+        resid, y, x = torch.randn(n, W, device=dev), rnd(n, W), rnd(n, W)
+        like = lambda: K.post_norm_residual(resid, y, wn, 1e-5, 0.0, kind="layer", layer_scale=ls, next_weight=nw, next_kind="layer")
+        lb = n * W * (8 + 2 * es)
+        add(f"tanh_norm_stream after a mixer ({name})", "post_norm_residual (layer norm, scale, next norm)",
+            lambda: K.tanh_norm_stream(resid, (nw, nb, alpha), y=y), nbytes=n * W * (8 + 2 * es), like_fn=like, like_bytes=lb)
+        add(f"tanh_norm_stream where a pass starts ({name}; embedding, step)", "post_norm_residual (layer norm, scale, next norm)",
+            lambda: K.tanh_norm_stream(resid, (nw, nb, alpha), y=y, embedding=(toks[:n], emb, 2.0), step=step),
+            nbytes=n * W * (8 + 3 * es), like_fn=like, like_bytes=lb)
+        ye, y2 = rnd(n, top, W), rnd(n, W)
+        ids = torch.stack([torch.randperm(E + I)[:top] for _ in range(n)]).int().to(dev)
+        wt = torch.rand(n, top, device=dev)
+        add(f"tanh_norm_stream after experts ({name}; {top} terms, identity experts, shared)",
+            "post_norm_residual (layer norm, scale, next norm)",
+            lambda: K.tanh_norm_stream(resid, (nw, nb, alpha), y=ye, routed=(ids, wt, E, x), addend=y2),
+            nbytes=n * W * (8 + (2 + top) * es), like_fn=like, like_bytes=lb)
+    # ---------------- attention whose values are its keys, beside attention over rows of keys and values
+    qn, kn = H * D, G * D
+    proj = rnd(T, 2 * qn + kn, s=0.5)
+    lproj = rnd(T, qn + 2 * kn, s=0.5)
+    col = K.key_factor_column(kn)
+    width = -(-(col + 2) // 8) * 8
+    pool, lpool = rnd(batch * (ctx + 1), width, s=0.5), rnd(batch * (ctx + 1), 2 * kn, s=0.5)
+    pool.view(torch.float32)[:, col // 2] = 1.0
+    tab = torch.arange(batch * (ctx + 1), dtype=torch.int32, device=dev).view(batch, ctx + 1)
+    rows_p = tab[:, :ctx].reshape(-1).contiguous()
+    pos_p = i32(list(range(prompt)) * batch)
+    qw, lqw, lkw = torch.rand(qn, device=dev) + 0.5, rnd(qn, s=0.1) + 1, rnd(kn, s=0.1) + 1
+    add("norm_query_keep_key", "attn_prepare (whole-row norms, query gain, keys and values)",
+        lambda: K.norm_query_keep_key(proj, pool, rows_p, pos_p, qn, kn, qw, 1e-6, 0.1, 256.0), nbytes=T * (2 * qn + 2 * kn) * es,
+        like_fn=lambda: K.attn_prepare(lproj, lpool, rows_p, pos_p, qn, kn, kn, lqw, lkw, 1e-6, 0.1, 256.0),
+        like_bytes=T * (2 * qn + 4 * kn) * es)
+    out = torch.empty(T, qn, dtype=dtype, device=dev)
+    gate = proj[:, qn + kn:]
+    scale = 1.0 / math.sqrt(D)
+    form = dict(v_col0=0, v_head_stride=D, key_factor_col=col, gate_elements=True)
+    flops = 4 * batch * H * D * prompt * (prompt + 1) / 2
+    add("attention on keys alone (prompts; score factor, element gate)", "attention on keys and values (prompts)",
+        lambda: K.sink_attention(out, proj, pool, tab, p_start, p_ctx, p_slot, None, batch, prompt, None, H, G, D, D, scale, 0.0,
+                                 gate=gate, **form), flops=flops,
+        like_fn=lambda: K.sink_attention(out, lproj, lpool, tab, p_start, p_ctx, p_slot, None, batch, prompt, None, H, G, D, D,
+                                         scale, 0.0))
+    for keys in (ctx + 1, 8193):
+        if keys != ctx + 1:
+            pool, lpool = rnd(batch * keys, width, s=0.5), rnd(batch * keys, 2 * kn, s=0.5)
+            pool.view(torch.float32)[:, col // 2] = 1.0
+        t2 = torch.arange(batch * keys, dtype=torch.int32, device=dev).view(batch, keys)
+        c2, (sp, per) = i32([keys - 1] * batch), split_plan(keys)
+        add(f"attention on keys alone (decode, {keys} keys; score factor, element gate)", "attention on keys and values (decode)",
+            lambda: K.sink_attention(out, proj, pool, t2, d_start, c2, p_slot, None, batch, 1, None, H, G, D, D, scale, 0.0,
+                                     num_splits=sp, split_keys=per, gate=gate, **form), nbytes=batch * keys * (kn * es + 4),
+            like_fn=lambda: K.sink_attention(out, lproj, lpool, t2, d_start, c2, p_slot, None, batch, 1, None, H, G, D, D, scale,
+                                             0.0, num_splits=sp, split_keys=per), like_bytes=batch * keys * 2 * kn * es)
+    # ---------------- latent attention beside the Pesivik path: its latent row is 96 + 32 columns
+    LD, pk, pr = kr + rot, 96, 32
+    PD = pk + pr
+    nq = H * (dim + rot)
+    lp = rnd(T, -(-nq // 8) * 8 + LD, s=0.5)
+    pp = rnd(T, -(-(qr + pk + pr + H) // 8) * 8, s=0.5)
+    lat_pool, pes_pool = rnd(batch * (ctx + 1), LD, s=0.5), rnd(batch * (ctx + 1), PD, s=0.5)
+    wkv, wq, pkv = rnd(kr, s=0.1) + 1, rnd(qr, s=0.1) + 1, rnd(pk, s=0.1) + 1
+    freqs, mag = K.rotary_frequencies(rot, 10000.0, *(V_SCALING[n] for n in ("factor", "original", "fast", "slow")))
+    fr = torch.tensor(freqs, dtype=torch.float64, device=dev)
+    cs, pcs = K.rope_table_freqs(pos_p, fr, mag), K.rope_table(pos_p, pr, 10000.0)
+    add("rope_table_freqs (interpolated, once per step)", "rope_table", lambda: K.rope_table_freqs(pos_p, fr, mag),
+        nbytes=T * (4 + rot * 4), like_fn=lambda: K.rope_table(pos_p, pr, 10000.0), like_bytes=T * (4 + pr * 4))
+    add("latent_prepare (no query latent, neighbour pairs)", "latent_prepare (query latent, halves)",
+        lambda: K.latent_prepare(lp[:, lp.shape[1] - LD:], lat_pool, rows_p, cs, None, wkv, 0, kr, rot, rot, 1e-6, "neighbours"),
+        nbytes=T * 2 * LD * es,
+        like_fn=lambda: K.latent_prepare(pp, pes_pool, rows_p, pcs, wq, pkv, qr, pk, pr, pr, 1e-6),
+        like_bytes=T * (2 * qr + 2 * PD) * es)
+    qa, pqa = torch.empty(T, H * LD, dtype=dtype, device=dev), torch.empty(T, H * PD, dtype=dtype, device=dev)
+    ukt, pukt = rnd(H, kr, dim, s=0.1), rnd(H, pk, dim, s=0.1)
+    add("head_linear (queries into the latent space)", "head_linear (Pesivik sizes)",
+        lambda: K.head_linear(qa, LD, lp, dim + rot, ukt), flops=2 * T * H * kr * dim,
+        like_fn=lambda: K.head_linear(pqa, PD, lp, dim + rot, pukt), like_flops=2 * T * H * pk * dim)
+    add("rope_heads (neighbour pairs)", "rope_heads (halves)",
+        lambda: K.rope_heads(qa[:, kr:], LD, lp[:, dim:], dim + rot, cs, H, rot, rot, "neighbours"), nbytes=T * H * rot * 2 * es,
+        like_fn=lambda: K.rope_heads(pqa[:, pk:], PD, lp[:, dim:], dim + rot, pcs, H, pr, pr), like_bytes=T * H * pr * 2 * es)
+    qa, pqa = rnd(T, H * LD, s=0.3), rnd(T, H * PD, s=0.3)
+    lat, plat = torch.empty(T, H * kr, dtype=dtype, device=dev), torch.empty(T, H * pk, dtype=dtype, device=dev)
+    pairs = batch * H * prompt * (prompt + 1)
+    add(f"attention over latent rows of {kr} + {rot} (prompts)", f"attention over latent rows of {pk} + {pr} (prompts)",
+        lambda: K.sink_attention(lat, qa, lat_pool, tab, p_start, p_ctx, p_slot, None, batch, prompt, None, H, 1, LD, kr, scale,
+                                 0.0, v_col0=0), flops=pairs * (LD + kr),
+        like_fn=lambda: K.sink_attention(plat, pqa, pes_pool, tab, p_start, p_ctx, p_slot, None, batch, prompt, None, H, 1, PD, pk,
+                                         scale, 0.0, v_col0=0), like_flops=pairs * (PD + pk))
+    for keys in (ctx + 1, 8193):
+        if keys != ctx + 1:
+            lat_pool, pes_pool = rnd(batch * keys, LD, s=0.5), rnd(batch * keys, PD, s=0.5)
+        t2 = torch.arange(batch * keys, dtype=torch.int32, device=dev).view(batch, keys)
+        c2, (sp, per) = i32([keys - 1] * batch), split_plan(keys)
+        add(f"attention over latent rows of {kr} + {rot} (decode, {keys} keys)", f"attention over latent rows of {pk} + {pr} (decode)",
+            lambda: K.sink_attention(lat, qa, lat_pool, t2, d_start, c2, p_slot, None, batch, 1, None, H, 1, LD, kr, scale, 0.0,
+                                     num_splits=sp, split_keys=per, v_col0=0), nbytes=batch * keys * LD * es,
+            like_fn=lambda: K.sink_attention(plat, pqa, pes_pool, t2, d_start, c2, p_slot, None, batch, 1, None, H, 1, PD, pk,
+                                             scale, 0.0, num_splits=sp, split_keys=per, v_col0=0), like_bytes=batch * keys * PD * es)
+    o, uv, puv = torch.empty(T, H * dim, dtype=dtype, device=dev), rnd(H, dim, kr, s=0.1), rnd(H, dim, pk, s=0.1)
+    add("head_linear (values out of the latent)", "head_linear (Pesivik sizes, head gate)",
+        lambda: K.head_linear(o, dim, lat, kr, uv), flops=2 * T * H * dim * kr,
+        like_fn=lambda: K.head_linear(o, dim, plat, pk, puv, pp[:, qr + PD:]), like_flops=2 * T * H * dim * pk)
+    # ---------------- feed-forward
+    gu = rnd(T, 2 * dff)
+    add("swiglu_scaled (gelu unit)", "swiglu_scaled (SiLU)", lambda: K.swiglu_scaled(gu[:, :dff], gu[:, dff:], form="gelu_tanh"),
+        nbytes=T * dff * 3 * es, like_fn=lambda: K.swiglu_scaled(gu[:, :dff], gu[:, dff:]))
+    del gu
+    x, router, corr = rnd(T, W, s=0.5), rnd(E + I, W, s=W ** -0.5), rnd(E + I, s=0.02)
+    prouter, pcorr = rnd(E, W, s=W ** -0.5), rnd(E, s=0.02)
+    kw = dict(scores="softmax", group_score="max")
+    add("route_sigmoid_groups (softmax, best of a group, identity experts)", "route_sigmoid_groups (sigmoid, two best of a group)",
+        lambda: K.route_sigmoid_groups(x, router, corr, top, sz["groups"], sz["keep"], **kw), flops=2 * T * (E + I) * W,
+        like_fn=lambda: K.route_sigmoid_groups(x, prouter, pcorr, top, sz["groups"], sz["keep"]), like_flops=2 * T * E * W)
+    wts, ids = K.route_sigmoid_groups(x, router, corr, top, sz["groups"], sz["keep"], **kw)
+    pw, pid = K.route_sigmoid_groups(x, prouter, pcorr, top, sz["groups"], sz["keep"])
+    wgu, wdn, wup = rnd(E, 2 * ff, W, s=W ** -0.5), rnd(E, W, ff, s=ff ** -0.5), rnd(E, ff, W, s=W ** -0.5)
+    for name, n in (("prompts", T), ("decode", batch)):
+        xn, wn, idn, pwn, pidn = x[:n], wts[:n].contiguous(), ids[:n].contiguous(), pw[:n].contiguous(), pid[:n].contiguous()
+        real = int((idn < E).sum())
+        used = len({e for e in idn.flatten().tolist() if e < E})
+        if name == "prompts":
+            cost = dict(flops=2 * real * 3 * ff * W, like_flops=2 * n * top * 2 * ff * W)
+        else:
+            cost = dict(nbytes=used * 3 * ff * W * es, like_bytes=len(set(pidn.flatten().tolist())) * 2 * ff * W * es)
+        add(f"grouped_experts, clamped unit, identity experts skipped ({name})", f"grouped_experts, ungated ({name})",
+            lambda: K.grouped_experts(xn, wgu, wdn, wn, idn, activation="clamped", gated=True, limit=7.0, reduce=False),
+            like_fn=lambda: K.grouped_experts(xn, wup, wdn, pwn, pidn), **cost)
+    return rows
+
+
 def run(args) -> None:
     from bench import ClockSampler, peaks
 
@@ -1318,7 +1543,8 @@ def run(args) -> None:
     table, steps, kernels = {"pesivik": (P_SIZES, pesivik_step_throughput, pesivik_kernel_table),
                              "tisosun": (T_SIZES, tisosun_step_throughput, tisosun_kernel_table),
                              "gofezen": (G_SIZES, gofezen_step_throughput, gofezen_kernel_table),
-                             "torutar": (U_SIZES, torutar_step_throughput, torutar_kernel_table)}.get(
+                             "torutar": (U_SIZES, torutar_step_throughput, torutar_kernel_table),
+                             "povilorn": (V_SIZES, povilorn_step_throughput, povilorn_kernel_table)}.get(
         args.design, (SIZES, step_throughput, kernel_table))
     result = {"design": args.design, "dtype": "bf16", "data": "synthetic ids, random weights", "peaks": {"hbm_gbs": hbm_gbs, "bf16_tflops": tflops, "source": src},
               "batch": args.batch, "prompt_len": args.prompt_len, "l2_policy": "256 MiB written between timed runs", "sizes": {}}
