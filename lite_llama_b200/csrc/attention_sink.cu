@@ -645,6 +645,8 @@ __global__ void __launch_bounds__(128) sink_attention_split_kernel(AttnArgs a) {
   const float inv_cap = a.softcap > 0.f ? 1.0f / a.softcap : 0.f;
   const bool vec_ok = (D % VEC == 0) && (Dv % VEC == 0) && (a.kv_stride % VEC == 0) && (a.v_col0 % VEC == 0) &&
                       (a.v_hstride % VEC == 0) && (((uintptr_t)a.kv % 16) == 0);
+  // accumulator j of a lane: neighbouring columns in pairs, one shared-memory load each
+  auto value_col = [&](int j) { return (j >> 1) * 64 + 2 * lane + (j & 1); };
   for (int k0 = key_lo + warp * 32; k0 < key_hi; k0 += 128) {
     const int nk = min(32, key_hi - k0);
     float factor = a.scale;                        // lane j: what multiplies key j's dot products
@@ -694,10 +696,15 @@ __global__ void __launch_bounds__(128) sink_attention_split_kernel(AttnArgs a) {
           const uint4 raw = *reinterpret_cast<const uint4*>(kr + d);
           const T* e = reinterpret_cast<const T*>(&raw);
 #pragma unroll
-          for (int c = 0; c < VEC; ++c) {
-            const float kvv = to_f32(e[c]);
+          for (int c = 0; c < VEC; c += 4) {
 #pragma unroll
-            for (int r = 0; r < kSplitRows; ++r) sc[r] = fmaf(qs[r * Dq + d + c], kvv, sc[r]);
+            for (int r = 0; r < kSplitRows; ++r) {
+              const float4 qv = *reinterpret_cast<const float4*>(qs + r * Dq + d + c);
+              sc[r] = fmaf(qv.x, to_f32(e[c]), sc[r]);
+              sc[r] = fmaf(qv.y, to_f32(e[c + 1]), sc[r]);
+              sc[r] = fmaf(qv.z, to_f32(e[c + 2]), sc[r]);
+              sc[r] = fmaf(qv.w, to_f32(e[c + 3]), sc[r]);
+            }
           }
         }
       } else {
@@ -727,9 +734,17 @@ __global__ void __launch_bounds__(128) sink_attention_split_kernel(AttnArgs a) {
     for (int kk = 0; kk < nk; ++kk) {
       float vv[DVJ];
 #pragma unroll
-      for (int j = 0; j < DVJ; ++j) {
-        const int d = lane + 32 * j;
-        vv[j] = d < Dv ? to_f32(vs[kk * vp + d]) : 0.f;
+      for (int j = 0; j < DVJ; j += 2) {
+        const int d = value_col(j);
+        if (vec_ok) {                              // Dv is even: both columns or none
+          struct alignas(2 * sizeof(T)) Pair { T a, b; } p = {};
+          if (d < Dv) p = *reinterpret_cast<const Pair*>(vs + kk * vp + d);
+          vv[j] = d < Dv ? to_f32(p.a) : 0.f;
+          vv[j + 1] = d < Dv ? to_f32(p.b) : 0.f;
+        } else {
+          vv[j] = d < Dv ? to_f32(vs[kk * vp + d]) : 0.f;
+          vv[j + 1] = d + 1 < Dv ? to_f32(vs[kk * vp + d + 1]) : 0.f;
+        }
       }
 #pragma unroll
       for (int r = 0; r < kSplitRows; ++r) {
@@ -746,7 +761,7 @@ __global__ void __launch_bounds__(128) sink_attention_split_kernel(AttnArgs a) {
     if (lane == 0) { dst[0] = m[r]; dst[1] = l[r]; }
 #pragma unroll
     for (int j = 0; j < DVJ; ++j) {
-      const int d = lane + 32 * j;
+      const int d = value_col(j);
       if (d < Dv) dst[2 + d] = acc[r][j];
     }
   }

@@ -43,8 +43,49 @@ __global__ void rope_table_kernel(float* __restrict__ cs, const int* __restrict_
   cs[t * dims + half + k] = s;
 }
 
-// One WARP per token (four tokens per CTA): the two statistics are warp reductions, nothing waits on a barrier.
-template <typename T>
+// RMS norm of `n` elements by one warp, src -> dst (may be the same); NV > 0: the elements stay in registers between the
+// statistic and the scaling, in 16-byte vectors (aligned rows, n a multiple of the vector, at most NV vectors a lane).
+template <typename T, int NV>
+__device__ __forceinline__ void warp_rms(T* __restrict__ dst, const T* __restrict__ src, const T* __restrict__ w, int n,
+                                         float eps, int lane) {
+  float ss = 0.f;
+  if constexpr (NV > 0) {
+    constexpr int V = 16 / (int)sizeof(T);
+    uint4 raw[NV], wr[NV];
+#pragma unroll
+    for (int u = 0; u < NV; ++u) {
+      const int i = (u * 32 + lane) * V;
+      raw[u] = wr[u] = make_uint4(0u, 0u, 0u, 0u);
+      if (i < n) { raw[u] = *reinterpret_cast<const uint4*>(src + i); wr[u] = *reinterpret_cast<const uint4*>(w + i); }
+    }
+#pragma unroll
+    for (int u = 0; u < NV; ++u) {
+      const T* e = reinterpret_cast<const T*>(&raw[u]);
+#pragma unroll
+      for (int c = 0; c < V; ++c) { const float v = to_f32(e[c]); ss = fmaf(v, v, ss); }
+    }
+    const float rstd = 1.0f / sqrtf(warp_reduce_sum(ss) / (float)n + eps);
+#pragma unroll
+    for (int u = 0; u < NV; ++u) {
+      const int i = (u * 32 + lane) * V;
+      const T* e = reinterpret_cast<const T*>(&raw[u]);
+      const T* we = reinterpret_cast<const T*>(&wr[u]);
+      uint4 res;
+      T* re = reinterpret_cast<T*>(&res);
+#pragma unroll
+      for (int c = 0; c < V; ++c) re[c] = from_f32<T>(to_f32(e[c]) * rstd * to_f32(we[c]));
+      if (i < n) *reinterpret_cast<uint4*>(dst + i) = res;
+    }
+  } else {
+    for (int i = lane; i < n; i += 32) { const float v = to_f32(src[i]); ss = fmaf(v, v, ss); }
+    const float rstd = 1.0f / sqrtf(warp_reduce_sum(ss) / (float)n + eps);
+    for (int i = lane; i < n; i += 32) dst[i] = from_f32<T>(to_f32(src[i]) * rstd * to_f32(w[i]));
+  }
+}
+
+// One WARP per token (four tokens per CTA): the two statistics are warp reductions, nothing waits on a barrier.  NV > 0:
+// the vector form of the latent norm.
+template <typename T, int NV>
 __global__ void __launch_bounds__(128) latent_prepare_kernel(T* __restrict__ proj, int64_t stride, T* __restrict__ pool,
                                                              int64_t pool_stride, const int* __restrict__ rows,
                                                              const float* __restrict__ cs_table,
@@ -59,16 +100,8 @@ __global__ void __launch_bounds__(128) latent_prepare_kernel(T* __restrict__ pro
   const T* b = a + q_rank;
   const T* r = b + kv_rank;
   T* dst = pool + (int64_t)rows[t] * pool_stride;
-  float ss = 0.f, rstd;
-  if (q_rank > 0) {
-    for (int i = lane; i < q_rank; i += 32) { const float v = to_f32(a[i]); ss = fmaf(v, v, ss); }
-    rstd = 1.0f / sqrtf(warp_reduce_sum(ss) / (float)q_rank + eps);
-    for (int i = lane; i < q_rank; i += 32) a[i] = from_f32<T>(to_f32(a[i]) * rstd * to_f32(wq[i]));
-  }
-  ss = 0.f;
-  for (int i = lane; i < kv_rank; i += 32) { const float v = to_f32(b[i]); ss = fmaf(v, v, ss); }
-  rstd = 1.0f / sqrtf(warp_reduce_sum(ss) / (float)kv_rank + eps);
-  for (int i = lane; i < kv_rank; i += 32) dst[i] = from_f32<T>(to_f32(b[i]) * rstd * to_f32(wkv[i]));
+  if (q_rank > 0) warp_rms<T, 0>(a, a, wq, q_rank, eps, lane);
+  warp_rms<T, NV>(dst, b, wkv, kv_rank, eps, lane);
   const int half = rot_dims / 2;
   const float* cs = cs_table + t * rot_dims;
   for (int i = lane; i < half; i += 32) {
@@ -135,9 +168,18 @@ extern "C" int b2l_latent_prepare(void* proj, int64_t proj_row_stride, void* poo
   if (tokens <= 0) return B2L_OK;
   cudaStream_t st = (cudaStream_t)stream;
   B2L_DISPATCH_FLOAT(dtype, "latent_prepare", {
-    b2l_launch(latent_prepare_kernel<T>, dim3((unsigned)cdiv64(tokens, 4)), dim3(128), (size_t)0, st, (T*)proj,
-               proj_row_stride, (T*)pool, pool_row_stride, (const int*)kv_rows_i32, (const float*)cos_sin_f32,
-               (const T*)q_norm_weight, (const T*)kv_norm_weight, tokens, q_rank, kv_rank, rot_dim, rot_dims, pairing, eps);
+    constexpr int VEC = 16 / (int)sizeof(T);
+    auto al = [](const void* p) { return (uintptr_t)p % 16 == 0; };
+    const bool vec = q_rank % VEC == 0 && kv_rank % VEC == 0 && proj_row_stride % VEC == 0 && pool_row_stride % VEC == 0 &&
+                     al(proj) && al(pool) && al(kv_norm_weight);
+    auto go = [&](auto kernel) {
+      b2l_launch(kernel, dim3((unsigned)cdiv64(tokens, 4)), dim3(128), (size_t)0, st, (T*)proj, proj_row_stride, (T*)pool,
+                 pool_row_stride, (const int*)kv_rows_i32, (const float*)cos_sin_f32, (const T*)q_norm_weight,
+                 (const T*)kv_norm_weight, tokens, q_rank, kv_rank, rot_dim, rot_dims, pairing, eps);
+    };
+    if (vec && kv_rank <= 32 * VEC) go(latent_prepare_kernel<T, 1>);
+    else if (vec && kv_rank <= 64 * VEC) go(latent_prepare_kernel<T, 2>);
+    else go(latent_prepare_kernel<T, 0>);
   });
   B2L_LAUNCH_CHECK();
   return B2L_OK;

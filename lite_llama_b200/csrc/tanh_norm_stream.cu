@@ -13,7 +13,6 @@
 // `experts` on are identity experts: they have no rows in y, their output is their input x times the weight.
 // With a row list (the output norm) only the listed tokens are read and the residual is not written.
 #include "common.cuh"
-#include "rowvec.cuh"
 
 namespace {
 
@@ -28,15 +27,38 @@ struct TanhStreamArgs {
   const int* rows; int64_t chunks, total;        // chunks of C elements per row; chunks of all rows
 };
 
+// C consecutive elements: 16-byte accesses of T (C = 8 for the 16-bit types, 4 for fp32; the fp32 residual then takes two
+// or one), or scalars (C = 1)
 template <int C, typename T>
 __device__ __forceinline__ void load_c(const T* p, float (&v)[C]) {
-  if constexpr (C == 4) row_load4(p, v);
-  else v[0] = to_f32(p[0]);
+  if constexpr (C == 1) {
+    v[0] = to_f32(p[0]);
+  } else {
+    constexpr int V = 16 / (int)sizeof(T);
+#pragma unroll
+    for (int i = 0; i < C; i += V) {
+      const uint4 raw = *reinterpret_cast<const uint4*>(p + i);
+      const T* e = reinterpret_cast<const T*>(&raw);
+#pragma unroll
+      for (int c = 0; c < V; ++c) v[i + c] = to_f32(e[c]);
+    }
+  }
 }
 template <int C, typename T>
 __device__ __forceinline__ void store_c(T* p, const float (&v)[C]) {
-  if constexpr (C == 4) row_store4(p, v);
-  else p[0] = from_f32<T>(v[0]);
+  if constexpr (C == 1) {
+    p[0] = from_f32<T>(v[0]);
+  } else {
+    constexpr int V = 16 / (int)sizeof(T);
+#pragma unroll
+    for (int i = 0; i < C; i += V) {
+      uint4 raw;
+      T* e = reinterpret_cast<T*>(&raw);
+#pragma unroll
+      for (int c = 0; c < V; ++c) e[c] = from_f32<T>(v[i + c]);
+      *reinterpret_cast<uint4*>(p + i) = raw;
+    }
+  }
 }
 template <int C, typename T>
 __device__ __forceinline__ void add_c(const T* p, float scale, float (&v)[C]) {
@@ -133,14 +155,14 @@ extern "C" int b2l_tanh_norm_stream(void* residual_f32, void* act, const void* y
   a.addend = addend; a.tokens = (const int*)tokens_i32; a.embed = embed; a.vocab = vocab; a.embed_scale = embed_scale;
   a.step = step; a.first = first; a.alpha = alpha; a.w = w; a.b = b; a.rows = (const int*)rows_i32;
   B2L_DISPATCH_FLOAT(dtype, "tanh_norm_stream", {
-    const bool vec = n % 4 == 0 && (!y || y_row_stride % 4 == 0) && (!x || x_row_stride % 4 == 0) &&
-                     row_aligned4<float>(residual_f32) && row_aligned4<T>(act) && row_aligned4<T>(y) && row_aligned4<T>(x) &&
-                     row_aligned4<T>(addend) && row_aligned4<T>(embed) && row_aligned4<T>(step) && row_aligned4<T>(w) &&
-                     row_aligned4<T>(b);
-    a.chunks = vec ? n / 4 : n;
+    constexpr int C = 16 / (int)sizeof(T);
+    auto al = [](const void* p) { return (uintptr_t)p % 16 == 0; };             // true for absent operands too
+    const bool vec = n % C == 0 && (!y || y_row_stride % C == 0) && (!x || x_row_stride % C == 0) && al(residual_f32) &&
+                     al(act) && al(y) && al(x) && al(addend) && al(embed) && al(step) && al(w) && al(b);
+    a.chunks = vec ? n / C : n;
     a.total = a.chunks * num_rows;
     const dim3 grid((unsigned)cdiv64(a.total, 256));
-    if (vec) b2l_launch(tanh_norm_stream_kernel<T, 4>, grid, dim3(256), (size_t)0, st, a);
+    if (vec) b2l_launch(tanh_norm_stream_kernel<T, C>, grid, dim3(256), (size_t)0, st, a);
     else b2l_launch(tanh_norm_stream_kernel<T, 1>, grid, dim3(256), (size_t)0, st, a);
   });
   B2L_LAUNCH_CHECK();
